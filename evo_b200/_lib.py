@@ -138,7 +138,7 @@ class SumNormParams(C.Structure):
     _fields_ = [("x", C.c_void_p), ("y", C.c_void_p * SUM_NORM_BRANCHES), ("ldy", C.c_int64 * SUM_NORM_BRANCHES),
                 ("norm_w", C.c_void_p * SUM_NORM_BRANCHES), ("scale", C.c_float * SUM_NORM_BRANCHES), ("n_branches", C.c_int),
                 ("eps", C.c_float), ("out", C.c_void_p * 2), ("w", C.c_void_p * 2), ("ldo", C.c_int64),
-                ("dtype", C.c_int), ("rows", C.c_int64), ("D", C.c_int), ("gather", C.c_void_p)]
+                ("dtype", C.c_int), ("rows", C.c_int64), ("D", C.c_int), ("gather", C.c_void_p), ("col_scale", C.c_void_p)]
 
 
 class ConvActParams(C.Structure):
@@ -195,6 +195,29 @@ class MlstmParams(C.Structure):
                 ("gate", C.c_void_p), ("ld_gate", C.c_int64), ("norm_w", C.c_void_p), ("eps", C.c_float),
                 ("state", C.c_void_p), ("mstate", C.c_void_p), ("zero_start", C.c_int),
                 ("out", C.c_void_p), ("ldo", C.c_int64), ("dtype", C.c_int),
+                ("B", C.c_int), ("L", C.c_int64), ("H", C.c_int), ("dk", C.c_int), ("dv", C.c_int)]
+
+
+class GluActParams(C.Structure):
+    _fields_ = [("gate", C.c_void_p), ("up", C.c_void_p), ("ld", C.c_int64), ("out", C.c_void_p), ("ldo", C.c_int64), ("rows", C.c_int64), ("F", C.c_int), ("act", C.c_int),
+                ("group_w", C.c_void_p), ("ldw", C.c_int64), ("group", C.c_int), ("n_groups", C.c_int), ("tail_w", C.c_int),
+                ("dtype", C.c_int), ("limit", C.c_float), ("slope", C.c_float)]
+
+
+class MixedAttnParams(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("q_tok_stride", C.c_int64),
+                ("k", C.c_void_p), ("v", C.c_void_p), ("k_tok_stride", C.c_int64), ("v_tok_stride", C.c_int64),
+                ("k_batch_stride", C.c_int64), ("v_batch_stride", C.c_int64),
+                ("gate", C.c_void_p), ("gate_tok_stride", C.c_int64), ("temp", C.c_void_p), ("talk", C.c_void_p),
+                ("out", C.c_void_p), ("ldo", C.c_int64), ("dtype", C.c_int),
+                ("B", C.c_int), ("Lq", C.c_int64), ("H", C.c_int), ("G", C.c_int), ("dk", C.c_int), ("dv", C.c_int),
+                ("q_pos0", C.c_int64), ("pos_dev", C.c_void_p), ("max_keys", C.c_int64), ("chunk", C.c_int64), ("scale", C.c_float), ("cuda_cores", C.c_int)]
+
+
+class GlaParams(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("ld", C.c_int64), ("alpha", C.c_void_p), ("q_scale", C.c_float),
+                ("gate", C.c_void_p), ("ld_gate", C.c_int64), ("norm_w", C.c_void_p), ("eps", C.c_float),
+                ("state", C.c_void_p), ("zero_start", C.c_int), ("out", C.c_void_p), ("ldo", C.c_int64), ("dtype", C.c_int),
                 ("B", C.c_int), ("L", C.c_int64), ("H", C.c_int), ("dk", C.c_int), ("dv", C.c_int)]
 
 
@@ -272,6 +295,12 @@ SIGNATURES = {
     "evo_post_norm": (C.c_int, [C.POINTER(PostNormParams), C.c_void_p]),
     "evo_mlstm_workspace": (C.c_size_t, [C.POINTER(MlstmParams)]),
     "evo_mlstm_fwd": (C.c_int, [C.POINTER(MlstmParams), C.c_void_p, C.c_size_t, C.c_void_p]),
+    "evo_glu_act_ex": (C.c_int, [C.POINTER(GluActParams), C.c_void_p]),
+    "evo_mixed_attn_workspace": (C.c_size_t, [C.POINTER(MixedAttnParams)]),
+    "evo_mixed_attn_fwd": (C.c_int, [C.POINTER(MixedAttnParams), C.c_void_p, C.c_size_t, C.c_void_p]),
+    "evo_low_rank_decay": (C.c_int, [C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_float, C.c_void_p, C.c_int64, C.c_int, C.c_int, C.c_int, C.c_void_p]),
+    "evo_gla_workspace": (C.c_size_t, [C.POINTER(GlaParams)]),
+    "evo_gla_fwd": (C.c_int, [C.POINTER(GlaParams), C.c_void_p, C.c_size_t, C.c_void_p]),
     "evo_moe_route": (C.c_int, [C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int64, C.c_int, C.c_int, C.c_int, C.c_float, C.c_int, C.c_void_p]),
 }
 

@@ -15,7 +15,8 @@ LIB = os.path.join(HERE, "libevo_b200.so")
 SOURCES = ["api.cu", "elementwise.cu", "hyena.cu", "gemm_tcgen05.cu", "gemm_smallm.cu", "attention.cu", "attention_pp.cu", "decode.cu", "scoring.cu", "sampler.cu", "ingest.cu", "die_map.cu",
            "rowops.cu", "hgrn2.cu", "window_attention.cu", "window_attention_mma.cu", "gemm_simt.cu",
            "mingru.cu", "latent_attention.cu", "moe.cu",
-           "branch_ops.cu", "matrix_state.cu", "attention_prep.cu", "post_norm.cu"]
+           "branch_ops.cu", "matrix_state.cu", "attention_prep.cu", "post_norm.cu",
+           "mixed_attention.cu"]
 # comparators for the GPU tests (cuBLASLt GEMM, CUDA-core attention): a separate library, never loaded by the product
 TEST_SRC = os.path.join(HERE, "..", "tests", "support", "test_support.cu")
 TEST_LIB = os.path.join(HERE, "..", "tests", "support", "libevo_b200_test.so")
@@ -48,6 +49,9 @@ def build(force: bool = False, verbose: bool = False) -> str:
 
     def cc(src):
         obj = os.path.join(OBJ, os.path.basename(src).replace(".cu", ".o"))
+        odig, ostamp = _digest([src] + hdrs), obj + ".stamp"
+        if not force and os.path.exists(obj) and os.path.exists(ostamp) and open(ostamp).read() == odig:
+            return obj
         r = subprocess.run([NVCC, *FLAGS, "-c", src, "-o", obj], capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"nvcc failed on {src}:\n{r.stdout}\n{r.stderr}")
@@ -55,6 +59,8 @@ def build(force: bool = False, verbose: bool = False) -> str:
             sys.stderr.write(r.stderr)
         with open(obj + ".ptxas.log", "w") as f:
             f.write(r.stderr)
+        with open(ostamp, "w") as f:
+            f.write(odig)
         return obj
 
     with ThreadPoolExecutor(max_workers=min(8, len(srcs))) as ex:

@@ -84,11 +84,13 @@ __global__ void __launch_bounds__(256) sum_norm_kernel(evo_sum_norm_params p) {
     }
   }
   float* xr = p.x + src * D;
+  const bf16* cs = (const bf16*)p.col_scale;
   float ss = 0.f;
   if (VEC) {
     for (int c = tid * 4; c < D; c += nt * 4) {
-      float v[4], add[4] = {0.f, 0.f, 0.f, 0.f};
+      float v[4], add[4] = {0.f, 0.f, 0.f, 0.f}, cw[4];
       Vec4<float>::load(xr + c, v);
+      if (cs) Vec4<bf16>::load(cs + c, cw);
 #pragma unroll
       for (int b = 0; b < EVO_SUM_NORM_BRANCHES; ++b) {
         if (b < p.n_branches) {
@@ -105,7 +107,7 @@ __global__ void __launch_bounds__(256) sum_norm_kernel(evo_sum_norm_params p) {
         }
       }
 #pragma unroll
-      for (int u = 0; u < 4; ++u) { v[u] += add[u]; ss = fmaf(v[u], v[u], ss); }
+      for (int u = 0; u < 4; ++u) { v[u] = cs ? fmaf(cw[u], add[u], v[u]) : v[u] + add[u]; ss = fmaf(v[u], v[u], ss); }
       Vec4<float>::store(xs + c, v);
       if (p.n_branches > 0 && !p.gather) Vec4<float>::store(xr + c, v);
     }
@@ -121,7 +123,7 @@ __global__ void __launch_bounds__(256) sum_norm_kernel(evo_sum_norm_params p) {
         add = fmaf(p.scale[b], y, add);
       }
     }
-    v += add;
+    v = cs ? fmaf(__bfloat162float(cs[c]), add, v) : v + add;
     xs[c] = v;
     if (p.n_branches > 0 && !p.gather) xr[c] = v;
     ss = fmaf(v, v, ss);
@@ -385,6 +387,7 @@ extern "C" int evo_sum_norm(const evo_sum_norm_params* p, void* stream) {
     vec = vec && p->ldy[b] % 4 == 0 && (p->dtype ? aligned4<float>(p->y[b]) : aligned4<bf16>(p->y[b]));
     if (p->norm_w[b]) vec = vec && aligned4<bf16>(p->norm_w[b]);
   }
+  vec = vec && (!p->col_scale || aligned4<bf16>(p->col_scale));
   for (int n = 0; n < 2; ++n)
     if (p->out[n]) vec = vec && aligned4<bf16>(p->w[n]) && (p->dtype ? aligned4<float>(p->out[n]) : aligned4<bf16>(p->out[n]));
   auto kern = p->dtype ? (vec ? sum_norm_kernel<float, true> : sum_norm_kernel<float, false>) : (vec ? sum_norm_kernel<bf16, true> : sum_norm_kernel<bf16, false>);

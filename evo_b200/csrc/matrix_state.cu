@@ -1,6 +1,7 @@
 // Recurrences whose state is a (dk x dv) matrix per head, carried in fp32 registers for the whole call:
 //   gated delta rule   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q        (evo_gated_delta_fwd)
 //   state-space dual   S <- a S + (dt B) x^T;  y = S^T C + D x                             (evo_ssd_fwd)
+//   per-channel decay  S <- diag(a) S + k v^T;  o = S^T q                                (evo_gla_fwd)
 //   matrix memory      m' = max(f + m, i);  S <- e^{f+m-m'} S + e^{i-m'} k v^T;  n alike;  o = S^T q / (max(|n.q|, e^{-m'}) + c)   (evo_mlstm_fwd)
 // with everything around them that the recurrence consumes computed here in fp32 from the activated projections: the unit norms of
 // q and k, sigmoid / softplus / exponentials of the per-head gates, and for the delta rule the head's RMS norm, weight and SiLU gate.
@@ -24,6 +25,8 @@
 // with a, b the round's decay and input factors and P_t = a_0 .. a_t, so the warps take the round's k_s.q_t and n_0.q_t dot products from
 // the staged rows (one thread per pair), one thread per token folds them, and n_0 is advanced to the round's end the same way; every CTA of a head does this
 // for itself, so a head spread over several CTAs needs no exchange.
+// The per-channel decay is the state-space loop with one decay per state row, staged beside the (key, query) pairs, and the delta rule's
+// epilogue; evo_low_rank_decay computes the decays sigmoid(A2 u + b)^(1/tau) of all rows and channels beforehand, in fp32.
 // The single-token step is the same kernel with L == 1.
 #include "common.cuh"
 #include <stdlib.h>
@@ -50,7 +53,7 @@ __device__ __forceinline__ float warp_sum(float v) {
 }
 
 constexpr int TCH = 16;      // tokens staged per round
-enum { MODE_DELTA = 0, MODE_SSD = 1, MODE_MLSTM = 2 };
+enum { MODE_DELTA = 0, MODE_SSD = 1, MODE_MLSTM = 2, MODE_GLA = 3 };
 
 // what both recurrences look like to the time loop
 struct ScanArgs {
@@ -67,6 +70,7 @@ struct ScanArgs {
   // matrix memory: gate biases, soft cap, running maximum (B, H), and beside y the reciprocal denominators per (row, head);
   // a head's state is its dk x dv matrix followed by the dk entries of the normaliser
   const void* i_bias; const void* f_bias; float cap, den_eps; float* mstate; float* em;
+  const float* alpha;                                              // per-channel decay: (rows, H*dk)
 };
 
 // soft cap c tanh(z / c) (c <= 0: none) and log sigmoid
@@ -85,6 +89,7 @@ __global__ void __launch_bounds__(RPT <= 4 ? 1024 : (RPT <= 32 ? 512 : 256), 1) 
   float* nvec = os + TCH * dvp;                            // [dkp]        matrix memory: the normaliser at the round's start
   float* kqd = nvec + dkp;                                 // [TCH][TCH]   k_s . q_t (s <= t)
   float* n0q = kqd + TCH * TCH;                            // [TCH]        n_0 . q_t
+  float* al = nvec;                                        // [TCH][dkp]   per-channel decay (in the place of the matrix memory's arrays)
   const int h = blockIdx.x, b = blockIdx.y, g = h / (p.H / p.G);
   const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, nw = nthr >> 5;
   const int j0 = blockIdx.z * dvp;                         // first value channel of this CTA
@@ -95,8 +100,9 @@ __global__ void __launch_bounds__(RPT <= 4 ? 1024 : (RPT <= 32 ? 512 : 256), 1) 
   float* Sg = p.state ? p.state + ((int64_t)b * p.H + h) * dk * (int64_t)(MODE == MODE_MLSTM ? dv + 1 : dv) : nullptr;
   if (MODE == MODE_MLSTM)
     for (int e = tid; e < dkp; e += nthr) nvec[e] = (Sg && !p.zero_start && e < dk) ? Sg[(int64_t)dk * dv + e] : 0.f;
-  const float A = MODE == MODE_MLSTM ? 0.f : expf(__bfloat162float(((const bf16*)p.A_log)[h]));
-  const float dtb = MODE == MODE_MLSTM ? 0.f : __bfloat162float(((const bf16*)p.dt_bias)[h]);
+  constexpr bool HEAD_DECAY = MODE == MODE_DELTA || MODE == MODE_SSD;                     // decay from A_log, dt_bias and one number per token and head
+  const float A = !HEAD_DECAY ? 0.f : expf(__bfloat162float(((const bf16*)p.A_log)[h]));
+  const float dtb = !HEAD_DECAY ? 0.f : __bfloat162float(((const bf16*)p.dt_bias)[h]);
   float mrun = (MODE == MODE_MLSTM && p.mstate && !p.zero_start) ? p.mstate[(int64_t)b * p.H + h] : 0.f;      // thread 0's: the running maximum
   const float Dh = MODE == MODE_SSD ? __bfloat162float(((const bf16*)p.Dskip)[h]) : 0.f;
 
@@ -135,13 +141,14 @@ __global__ void __launch_bounds__(RPT <= 4 ? 1024 : (RPT <= 32 ? 512 : 256), 1) 
           sc[tt * 4 + 1] = 1.f / (1.f + expf(-bv));
           sc[tt * 4 + 2] = skq * rk * rq;
         }
-      } else if (MODE == MODE_MLSTM) {
+      } else if (MODE == MODE_MLSTM || MODE == MODE_GLA) {
         for (int e = lane; e < dkp; e += 32) {
           float2 o = make_float2(0.f, 0.f);
           if (e < dk) { o.x = ldf(kp + row * p.ld + e); o.y = ldf(qp + row * p.ld + e) * p.q_scale; }
           kq[tt * dkp + e] = o;
+          if (MODE == MODE_GLA) al[tt * dkp + e] = e < dk ? p.alpha[(row * p.H + h) * dk + e] : 0.f;
         }
-        if (lane == 0) {                                  // log forget gate, log input gate; the scan below turns them into factors
+        if (MODE == MODE_MLSTM && lane == 0) {                                  // log forget gate, log input gate; the scan below turns them into factors
           const float gi = ldf((const T*)p.s0 + row * p.lds + h) + __bfloat162float(((const bf16*)p.i_bias)[h]);
           const float gf = ldf((const T*)p.s1 + row * p.lds + h) + __bfloat162float(((const bf16*)p.f_bias)[h]);
           sc[tt * 4 + 0] = log_sigmoid(soft_cap(gf, p.cap));
@@ -222,7 +229,7 @@ __global__ void __launch_bounds__(RPT <= 4 ? 1024 : (RPT <= 32 ? 512 : 256), 1) 
       float v[CPT];
 #pragma unroll
       for (int c = 0; c < CPT; ++c) v[c] = vs[tt * dvp + jl + c];
-      const float dec = sc[tt * 4 + 0];
+      const float dec = MODE == MODE_GLA ? 0.f : sc[tt * 4 + 0];
       const float4* e = reinterpret_cast<const float4*>(kq + tt * dkp) + l;             // two state rows per 16-byte read; pair r at e[r * LPC]
       if (MODE == MODE_DELTA) {
         constexpr bool KEEP = RPT <= 16;                   // the keys stay in registers for the update, or are read again
@@ -276,17 +283,18 @@ __global__ void __launch_bounds__(RPT <= 4 ? 1024 : (RPT <= 32 ? 512 : 256), 1) 
 #pragma unroll
         for (int r = 0; r < RPT / 2; ++r) {
           const float4 f = e[r * LPC];
+          const float2 d2 = MODE == MODE_GLA ? reinterpret_cast<const float2*>(al + tt * dkp)[r * LPC + l] : make_float2(dec, dec);
 #pragma unroll
           for (int c = 0; c < CPT; ++c) {
-            S[c][2 * r] = fmaf(dec, S[c][2 * r], f.x * v[c]);          y[c] = fmaf(S[c][2 * r], f.y, y[c]);
-            S[c][2 * r + 1] = fmaf(dec, S[c][2 * r + 1], f.z * v[c]);  y[c] = fmaf(S[c][2 * r + 1], f.w, y[c]);
+            S[c][2 * r] = fmaf(d2.x, S[c][2 * r], f.x * v[c]);          y[c] = fmaf(S[c][2 * r], f.y, y[c]);
+            S[c][2 * r + 1] = fmaf(d2.y, S[c][2 * r + 1], f.z * v[c]);  y[c] = fmaf(S[c][2 * r + 1], f.w, y[c]);
           }
         }
 #pragma unroll
         for (int o = 1; o < LPC; o <<= 1)
 #pragma unroll
           for (int c = 0; c < CPT; ++c) y[c] += __shfl_xor_sync(0xffffffffu, y[c], o);
-        if (MODE == MODE_MLSTM) {
+        if (MODE == MODE_MLSTM || MODE == MODE_GLA) {
 #pragma unroll
           for (int c = 0; c < CPT; ++c)
             if (l == 0) {
@@ -320,7 +328,7 @@ __global__ void __launch_bounds__(RPT <= 4 ? 1024 : (RPT <= 32 ? 512 : 256), 1) 
           for (int64_t c = (int64_t)p.H * dv + lane; c < p.ldo; c += 32) stf(orow + c, 0.f);
       }
     }
-    if (MODE == MODE_DELTA && !p.y) {
+    if ((MODE == MODE_DELTA || MODE == MODE_GLA) && !p.y) {
       __syncthreads();
       // head norm, weight, SiLU gate, store: one warp per token
       const bf16* nwt = (const bf16*)p.norm_w;
@@ -357,7 +365,7 @@ __global__ void __launch_bounds__(RPT <= 4 ? 1024 : (RPT <= 32 ? 512 : 256), 1) 
   }
 }
 
-// head norm, weight and SiLU gate of the delta rule's read-outs when a head was spread over several CTAs: one warp per (row, head)
+// head norm, weight and SiLU gate of the delta rule's and the per-channel decay's read-outs when a head was spread over several CTAs: one warp per (row, head)
 template <typename T>
 __global__ void __launch_bounds__(256) delta_head_norm_kernel(ScanArgs p) {
   const int64_t wid = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -430,14 +438,15 @@ inline Plan plan(int dk, int dv, int64_t ctas, int64_t L) {
 
 template <typename T, int RPT, int LPC, int MODE>
 int launch(const ScanArgs& a, const Plan& pl, cudaStream_t st, const char* what) {
-  const size_t smem = sizeof(float) * ((size_t)2 * TCH * LPC * RPT + (size_t)2 * TCH * pl.dvc + (size_t)TCH * 4 + (size_t)LPC * RPT + (size_t)TCH * TCH + TCH);
+  const size_t smem = sizeof(float) * ((size_t)2 * TCH * LPC * RPT + (size_t)2 * TCH * pl.dvc + (size_t)TCH * 4 +
+                                       (MODE == MODE_GLA ? (size_t)TCH * LPC * RPT : (size_t)LPC * RPT + (size_t)TCH * TCH + TCH));
   auto kern = matrix_state_kernel<T, RPT, LPC, MODE>;
   if (smem > 48 * 1024) EVO_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   kern<<<dim3(a.H, a.B, pl.chunks), dim3(LPC * pl.dvc / columns_per_thread(RPT)), smem, st>>>(a, pl.dvc);
   int rc = check_launch(what);
   if (rc || MODE == MODE_SSD || !a.y) return rc;
   const int64_t warps = (int64_t)a.B * a.L * a.H;
-  if (MODE == MODE_DELTA) delta_head_norm_kernel<T><<<(unsigned)((warps + 7) / 8), 256, 0, st>>>(a);
+  if (MODE == MODE_DELTA || MODE == MODE_GLA) delta_head_norm_kernel<T><<<(unsigned)((warps + 7) / 8), 256, 0, st>>>(a);
   else mlstm_head_norm_kernel<T><<<(unsigned)((warps + 7) / 8), 256, 0, st>>>(a);
   return check_launch(what);
 }
@@ -535,4 +544,73 @@ extern "C" int evo_mlstm_fwd(const evo_mlstm_params* p, void* workspace, size_t 
   const ScanArgs a = mlstm_args(p);
   return p->dtype ? dispatch<float, MODE_MLSTM>(a, workspace, workspace_bytes, (cudaStream_t)stream, "evo_mlstm_fwd")
                   : dispatch<bf16, MODE_MLSTM>(a, workspace, workspace_bytes, (cudaStream_t)stream, "evo_mlstm_fwd");
+}
+
+// ---- per-channel decay: alpha[row, c] = sigmoid(sum_r a2[c, r] u[row, r] + bias[c]) ^ inv_tau.  A thread owns a channel, its CTA DT rows.
+namespace {
+constexpr int DT = 16;
+template <typename T>
+__global__ void __launch_bounds__(256) low_rank_decay_kernel(const T* __restrict__ u, int64_t ldu, const bf16* __restrict__ a2, const bf16* __restrict__ bias, float inv_tau,
+                                                             float* __restrict__ alpha, int64_t rows, int rank, int C) {
+  extern __shared__ __align__(16) float us[];               // [DT][r4]
+  const int r4 = (rank + 3) / 4 * 4;
+  const int64_t row0 = (int64_t)blockIdx.x * DT;
+  const int nt = (int)min((int64_t)DT, rows - row0);
+  for (int i = threadIdx.x; i < DT * r4; i += blockDim.x) {
+    const int t = i / r4, r = i % r4;
+    us[i] = (t < nt && r < rank) ? ldf(u + (row0 + t) * ldu + r) : 0.f;
+  }
+  __syncthreads();
+  const int c = blockIdx.y * blockDim.x + threadIdx.x;
+  if (c >= C) return;
+  float acc[DT];
+  const float b = __bfloat162float(bias[c]);
+#pragma unroll
+  for (int t = 0; t < DT; ++t) acc[t] = b;
+  const bf16* w = a2 + (int64_t)c * rank;
+  for (int r = 0; r < r4; r += 4) {
+    float wv[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) wv[k] = r + k < rank ? __bfloat162float(w[r + k]) : 0.f;
+#pragma unroll
+    for (int t = 0; t < DT; ++t) {
+      const float4 v = *reinterpret_cast<const float4*>(us + t * r4 + r);
+      acc[t] = fmaf(wv[0], v.x, fmaf(wv[1], v.y, fmaf(wv[2], v.z, fmaf(wv[3], v.w, acc[t]))));
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < DT; ++t)
+    if (t < nt) alpha[(row0 + t) * C + c] = expf(log_sigmoid(acc[t]) * inv_tau);
+}
+}  // namespace
+
+extern "C" int evo_low_rank_decay(const void* u, int64_t ldu, const void* a2, const void* bias, float inv_tau, float* alpha, int64_t rows, int rank, int channels, int dtype,
+                                  void* stream) {
+  EVO_REQUIRE(u && a2 && bias && alpha && rank > 0 && channels > 0 && ldu >= rank && rows >= 0, "evo_low_rank_decay: bad arguments");
+  const size_t smem = sizeof(float) * DT * (size_t)((rank + 3) / 4 * 4);
+  EVO_REQUIRE(smem <= 48 * 1024, "evo_low_rank_decay: rank (%d) must be at most 768", rank);
+  EVO_REQUIRE((channels + 255) / 256 <= 65535, "evo_low_rank_decay: too many channels");
+  if (rows == 0) return 0;
+  const dim3 grid((unsigned)((rows + DT - 1) / DT), (unsigned)((channels + 255) / 256));
+  if (dtype) low_rank_decay_kernel<float><<<grid, 256, smem, (cudaStream_t)stream>>>((const float*)u, ldu, (const bf16*)a2, (const bf16*)bias, inv_tau, alpha, rows, rank, channels);
+  else low_rank_decay_kernel<bf16><<<grid, 256, smem, (cudaStream_t)stream>>>((const bf16*)u, ldu, (const bf16*)a2, (const bf16*)bias, inv_tau, alpha, rows, rank, channels);
+  return check_launch("evo_low_rank_decay");
+}
+
+extern "C" size_t evo_gla_workspace(const evo_gla_params* p) {
+  const Plan pl = plan(p->dk, p->dv, (int64_t)p->B * p->H, p->L);
+  return pl.chunks > 1 ? sizeof(float) * (size_t)p->B * p->L * p->H * p->dv : 0;
+}
+
+extern "C" int evo_gla_fwd(const evo_gla_params* p, void* workspace, size_t workspace_bytes, void* stream) {
+  EVO_REQUIRE(p->q && p->k && p->v && p->alpha && p->gate && p->norm_w && p->out, "evo_gla_fwd: null argument");
+  EVO_REQUIRE(p->B >= 0 && p->L >= 0 && p->H > 0 && p->dk > 0 && p->dv > 0 && p->ldo >= (int64_t)p->H * p->dv, "evo_gla_fwd: bad shape");
+  if (p->B == 0 || p->L == 0) return 0;
+  ScanArgs a = {};
+  a.kk = p->k; a.qq = p->q; a.vv = p->v; a.ld = p->ld; a.alpha = p->alpha; a.q_scale = p->q_scale;
+  a.state = p->state; a.zero_start = p->zero_start;
+  a.gate = p->gate; a.ldg = p->ld_gate; a.norm_w = p->norm_w; a.eps = p->eps; a.out = p->out; a.ldo = p->ldo;
+  a.B = p->B; a.L = p->L; a.H = p->H; a.G = p->H; a.dk = p->dk; a.dv = p->dv;
+  return p->dtype ? dispatch<float, MODE_GLA>(a, workspace, workspace_bytes, (cudaStream_t)stream, "evo_gla_fwd")
+                  : dispatch<bf16, MODE_GLA>(a, workspace, workspace_bytes, (cudaStream_t)stream, "evo_gla_fwd");
 }

@@ -553,13 +553,20 @@ __device__ __forceinline__ float act_value(float z, int act) {
   if (act == 2) return 0.5f * z * (1.f + erff(z * 0.7071067811865476f));     // erf form of gelu
   return z * sigm<T>(z);                   // silu
 }
+// both factors of an element; act 3: the gate cut at `limit` with a steeper sigmoid, times the up value cut to [-limit, limit] plus one
+template <typename T>
+__device__ __forceinline__ float glu_value(float z, float u, int act, float limit, float slope) {
+  if (act == 3) { const float c = fminf(z, limit); return c * sigm<T>(slope * c) * (fminf(fmaxf(u, -limit), limit) + 1.f); }
+  return act_value<T>(z, act) * u;
+}
 
 // out[r, c] = act(g[r, c]) * u[r, c] * w(r, c) for c < F, zero for F <= c < ldo (u == nullptr: no second factor);
 // w = group_w[r * ldw + c / group] for c < n_groups * group, after them group_w[r * ldw + n_groups] with tail_w, else 1.
 // grid (rows, column chunks): few rows (a decoding step) still fill the GPU.  VEC: 4 columns per thread (F, group, strides multiples of 4).
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) glu_act_kernel(const T* __restrict__ g, const T* __restrict__ u, int64_t ld, T* __restrict__ out, int64_t ldo,
-                                                      int F, int act, const float* __restrict__ group_w, int64_t ldw, int group, int n_groups, int tail_w) {
+                                                      int F, int act, const float* __restrict__ group_w, int64_t ldw, int group, int n_groups, int tail_w,
+                                                      float limit, float slope) {
   const int64_t r = blockIdx.x;
   const T* gr = g + r * ld; const T* ur = u ? u + r * ld : nullptr;
   T* orow = out + r * ldo;
@@ -576,10 +583,10 @@ __global__ void __launch_bounds__(256) glu_act_kernel(const T* __restrict__ g, c
     if (wt != 0.f) {
       if (VEC) {
         const float4 g4 = ld4(gr + c), u4 = ur ? ld4(ur + c) : make_float4(1.f, 1.f, 1.f, 1.f);
-        v[0] = act_value<T>(g4.x, act) * u4.x * wt; v[1] = act_value<T>(g4.y, act) * u4.y * wt;
-        v[2] = act_value<T>(g4.z, act) * u4.z * wt; v[3] = act_value<T>(g4.w, act) * u4.w * wt;
+        v[0] = glu_value<T>(g4.x, u4.x, act, limit, slope) * wt; v[1] = glu_value<T>(g4.y, u4.y, act, limit, slope) * wt;
+        v[2] = glu_value<T>(g4.z, u4.z, act, limit, slope) * wt; v[3] = glu_value<T>(g4.w, u4.w, act, limit, slope) * wt;
       } else {
-        v[0] = act_value<T>(ldf(gr + c), act) * (ur ? ldf(ur + c) : 1.f) * wt;
+        v[0] = glu_value<T>(ldf(gr + c), ur ? ldf(ur + c) : 1.f, act, limit, slope) * wt;
       }
     }
   }
@@ -623,25 +630,34 @@ extern "C" int evo_branch_norm(const evo_branch_norm_params* p, void* stream) {
   return check_launch("evo_branch_norm");
 }
 
+extern "C" int evo_glu_act_ex(const evo_glu_act_params* p, void* stream) {
+  EVO_REQUIRE(p->gate && p->out && p->F > 0 && p->ldo >= p->F && p->act >= 0 && p->act <= 3, "evo_glu_act: bad arguments");
+  EVO_REQUIRE(p->act != 3 || (p->up && p->limit > 0.f), "evo_glu_act: the limited form needs both factors and a positive limit");
+  EVO_REQUIRE(p->group_w == nullptr || (p->group > 0 && p->n_groups > 0 && p->ldw >= p->n_groups + (p->tail_w ? 1 : 0)), "evo_glu_act: bad groups");
+  if (p->rows == 0) return 0;
+  const int av = p->dtype ? 16 : 8;
+  const bool vec = p->F % 4 == 0 && p->ld % 4 == 0 && p->ldo % 4 == 0 && (p->group_w == nullptr || (p->group % 4 == 0)) && aligned_to(p->gate, av) && aligned_to(p->up, av) &&
+                   aligned_to(p->out, av);
+  const int per = 256 * (vec ? 4 : 1);
+  EVO_REQUIRE((p->ldo + per - 1) / per <= 65535, "evo_glu_act: row too wide");
+  dim3 grid((unsigned)p->rows, (unsigned)((p->ldo + per - 1) / per)), block(256);
+  cudaStream_t st = (cudaStream_t)stream;
+#define EVO_GLU(TT, V) \
+  glu_act_kernel<TT, V><<<grid, block, 0, st>>>((const TT*)p->gate, (const TT*)p->up, p->ld, (TT*)p->out, p->ldo, p->F, p->act, p->group_w, p->ldw, p->group, p->n_groups, \
+                                                p->tail_w, p->limit, p->slope)
+  if (p->dtype) { if (vec) EVO_GLU(float, true); else EVO_GLU(float, false); }
+  else { if (vec) EVO_GLU(bf16, true); else EVO_GLU(bf16, false); }
+#undef EVO_GLU
+  return check_launch("evo_glu_act");
+}
+
 extern "C" int evo_glu_act(const void* gate, const void* up, int64_t ld, void* out, int64_t ldo, int64_t rows, int F, int act,
                            const float* group_w, int64_t ldw, int group, int n_groups, int tail_w, int dtype, void* stream) {
-  EVO_REQUIRE(gate && out && F > 0 && ldo >= F && act >= 0 && act <= 2, "evo_glu_act: bad arguments");
-  EVO_REQUIRE(group_w == nullptr || (group > 0 && n_groups > 0 && ldw >= n_groups + (tail_w ? 1 : 0)), "evo_glu_act: bad groups");
-  if (rows == 0) return 0;
-  const int av = dtype ? 16 : 8;
-  const bool vec = F % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 && (group_w == nullptr || (group % 4 == 0)) && aligned_to(gate, av) && aligned_to(up, av) && aligned_to(out, av);
-  const int per = 256 * (vec ? 4 : 1);
-  EVO_REQUIRE((ldo + per - 1) / per <= 65535, "evo_glu_act: row too wide");
-  dim3 grid((unsigned)rows, (unsigned)((ldo + per - 1) / per)), block(256);
-  cudaStream_t st = (cudaStream_t)stream;
-  if (dtype) {
-    if (vec) glu_act_kernel<float, true><<<grid, block, 0, st>>>((const float*)gate, (const float*)up, ld, (float*)out, ldo, F, act, group_w, ldw, group, n_groups, tail_w);
-    else glu_act_kernel<float, false><<<grid, block, 0, st>>>((const float*)gate, (const float*)up, ld, (float*)out, ldo, F, act, group_w, ldw, group, n_groups, tail_w);
-  } else {
-    if (vec) glu_act_kernel<bf16, true><<<grid, block, 0, st>>>((const bf16*)gate, (const bf16*)up, ld, (bf16*)out, ldo, F, act, group_w, ldw, group, n_groups, tail_w);
-    else glu_act_kernel<bf16, false><<<grid, block, 0, st>>>((const bf16*)gate, (const bf16*)up, ld, (bf16*)out, ldo, F, act, group_w, ldw, group, n_groups, tail_w);
-  }
-  return check_launch("evo_glu_act");
+  EVO_REQUIRE(act <= 2, "evo_glu_act: bad arguments");
+  evo_glu_act_params p = {};
+  p.gate = gate; p.up = up; p.ld = ld; p.out = out; p.ldo = ldo; p.rows = rows; p.F = F; p.act = act;
+  p.group_w = group_w; p.ldw = ldw; p.group = group; p.n_groups = n_groups; p.tail_w = tail_w; p.dtype = dtype;
+  return evo_glu_act_ex(&p, stream);
 }
 
 extern "C" int evo_scale_logits(const void* in, int64_t ldi, float* out, int64_t rows, int V, float mul, int dtype, void* stream) {

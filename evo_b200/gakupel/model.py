@@ -27,7 +27,7 @@ import os
 import torch
 
 from .. import _lib
-from .._lib import MlstmParams, MoeRouteParams, PostNormParams, QkPrepParams, WindowAttnParams, check, ptr
+from .._lib import MlstmParams, PostNormParams, QkPrepParams, WindowAttnParams, check, ptr
 from ..stream_model import StreamDecoder, _Packed, _round_up
 from .config import GakupelConfig
 
@@ -220,13 +220,8 @@ class Gakupel(StreamDecoder):
         """Routing weights (M, experts [+ 1: the always-on expert's gate]) fp32 from the stream's rows h."""
         pk = self._packed["layers"][i]
         n_extra = 1 if f.shared_ff else 0
-        route = torch.empty(M, f.experts + n_extra, dtype=torch.float32, device=h.device)
-        rp = MoeRouteParams(h=h.data_ptr(), ldh=h.shape[1], router_w=pk["router"].data_ptr(), correction=self.weights[f"l{i}.mlp.correction"].data_ptr(),
-                            weights=route.data_ptr(), ldw=f.experts + n_extra, chosen=chosen.data_ptr() if chosen is not None else None,
-                            rows=M, D=self.config.width, E=f.experts, top=f.top, n_extra=n_extra, score_fn=1, groups=f.groups, keep=f.keep,
-                            normalize=1, norm_eps=1e-20, scale=f.router_scale, dtype=self._dt)
-        self._record("moe_route", float(M) * self.config.width * h.element_size(), lambda: check(_lib.lib().evo_moe_route_ex(C.byref(rp), self._stream()), "evo_moe_route"))
-        return route
+        return self._moe_route(h, M, pk["router"], f.experts, f.top, correction=self.weights[f"l{i}.mlp.correction"], chosen=chosen, n_extra=n_extra,
+                               score_fn=1, groups=f.groups, keep=f.keep, normalize=1, norm_eps=1e-20, scale=f.router_scale)
 
     def _experts_sparse(self, i, f, h, M):
         """Only the chosen experts (see StreamDecoder._run_chosen_experts), then the weighted sum per token on top of the gated always-on expert."""

@@ -218,3 +218,8 @@ def load_named_tensors(model_dir: str, device, shapes: Dict[str, tuple], what: s
     if device.type == "cuda":
         torch.cuda.synchronize(device)
     return out, {"tensors": len(out), "bytes": nbytes}
+
+
+def stored_shapes(model_dir: str) -> Dict[str, tuple]:
+    """{tensor name: shape} of a checkpoint folder, from the files' headers."""
+    return {name: shape for path in shard_files(model_dir) for name, _, shape, _ in iter_safetensors(path)}

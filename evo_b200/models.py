@@ -99,9 +99,11 @@ def load_checkpoint(model_name: str = "evo-1-8k-base", config_path: Optional[str
 
 def _load_flat(family, model_dir: str, config: dict, device, dtype):
     """Families described by a flat table of checkpoint tensors (StreamDecoder subclasses)."""
-    from .ingest import load_named_tensors
+    from .ingest import load_named_tensors, stored_shapes
     cls, cfg_cls = family()
-    model = cls(cfg_cls.from_dict(config), dtype=dtype or torch.bfloat16)
+    # sizes that only a tensor's shape gives are read from the files' headers
+    extra = {"shapes": stored_shapes(model_dir)} if getattr(cfg_cls, "needs_shapes", False) else {}
+    model = cls(cfg_cls.from_dict(config, **extra), dtype=dtype or torch.bfloat16)
     dev = torch.device(device) if device is not None else torch.device("cpu")
     shapes = {k: tuple(v.shape) for k, v in model.weights.items()}
     tensors, model.ingest_stats = load_named_tensors(model_dir, dev, shapes, type(model).__name__, ignorable=getattr(model.config, "unused_tensor_names", ()))
@@ -139,6 +141,13 @@ def _load_gakupel(model_dir: str, config: dict, device, dtype, **kwargs):
     return _load_flat(family, model_dir, config, device, dtype)
 
 
+def _load_gagotar(model_dir: str, config: dict, device, dtype, **kwargs):
+    def family():
+        from .gagotar import Gagotar, GagotarConfig
+        return Gagotar, GagotarConfig
+    return _load_flat(family, model_dir, config, device, dtype)
+
+
 def _load_stripedhyena(model_dir: str, config: dict, device, dtype, model_name: str = "evo-1-8k-base", **kwargs):
     if dtype not in (None, torch.bfloat16):
         raise NotImplementedError("StripedHyena runs in bfloat16 (fp32 poles and residues) only")
@@ -151,6 +160,7 @@ ARCHITECTURES = {
     "Movalorn": (_load_movalorn, (torch.bfloat16, torch.float32)),
     "Nelovik": (_load_nelovik, (torch.bfloat16, torch.float32)),
     "Gakupel": (_load_gakupel, (torch.bfloat16, torch.float32)),
+    "Gagotar": (_load_gagotar, (torch.bfloat16, torch.float32)),
     "StripedHyena": (_load_stripedhyena, (torch.bfloat16,)),
     "StripedHyenaModelForCausalLM": (_load_stripedhyena, (torch.bfloat16,)),
 }

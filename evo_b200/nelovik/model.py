@@ -22,7 +22,7 @@ from typing import Optional
 import torch
 
 from .. import _lib
-from .._lib import QkPrepParams, SsdParams, SumNormParams, WindowAttnParams, check, ptr
+from .._lib import QkPrepParams, SsdParams, WindowAttnParams, check, ptr
 from ..stream_model import StreamDecoder, _Packed, _round_up
 from .config import NelovikConfig
 
@@ -104,19 +104,6 @@ class Nelovik(StreamDecoder):
         return cache.shape[1]
 
     # ---- kernels ---------------------------------------------------------------------------------
-    def _sum_norm(self, x, branches, outs, rows, gather=None):
-        """x += sum of the branches (y, ldy, norm weight or None, scale); outs: [(buffer, weight)] normed copies of the new x."""
-        cfg = self.config
-        p = SumNormParams(x=x.data_ptr(), n_branches=len(branches), eps=cfg.eps, dtype=self._dt, rows=rows, D=cfg.width,
-                          gather=gather.data_ptr() if gather is not None else None, ldo=_round_up(cfg.width, 64))
-        for b, (y, ldy, nw, scale) in enumerate(branches):
-            p.y[b], p.ldy[b], p.norm_w[b], p.scale[b] = y.data_ptr(), ldy, (nw.data_ptr() if nw is not None else None), scale
-        for n, (o, wt) in enumerate(outs):
-            p.out[n], p.w[n] = o.data_ptr(), wt.data_ptr()
-        esz = 4 if self._dt else 2
-        nbytes = rows * cfg.width * (8.0 + esz * (len(branches) + len(outs)))
-        self._record("sum_norm", nbytes, lambda: check(_lib.lib().evo_sum_norm(C.byref(p), self._stream()), "evo_sum_norm"))
-
     def _delta(self, r, i, m, h, B, L, rec, fresh):
         y, ld = self._delta_mixer(r, i, m, h, B, L, rec, fresh)
         return [(y, ld, None, 1.0)]

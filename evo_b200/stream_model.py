@@ -1,5 +1,5 @@
 """Shared base of the model families that keep the residual stream in fp32 and are described by a flat table of checkpoint
-tensors (Zaverax, Movalorn, Nelovik): weight holding and strict loading, the padded GEMM weights, the linear-layer dispatch
+tensors (Zaverax, Movalorn, Nelovik, Gakupel, Gagotar): weight holding and strict loading, the padded GEMM weights, the linear-layer dispatch
 (tcgen05 GEMMs for bf16 activations, the CUDA-core fp32 GEMM for the all-fp32 mode), the inference-state holders, the
 forward protocol and the on-device generation loop.  A family provides `_ensure_packed()` and
 `_body(ids, B, L, state, offset, pos_dev=None, rows=None) -> fp32 logits`; everything that drives a model -- the generation loop,
@@ -23,7 +23,7 @@ import torch
 import torch.nn as nn
 
 from . import _lib
-from ._lib import EPI_NONE, ConvActParams, GatedDeltaParams, check, ptr
+from ._lib import EPI_NONE, ConvActParams, GatedDeltaParams, GluActParams, MoeRouteParams, SumNormParams, check, ptr
 from .engine import KernelOps
 from .stripedhyena.cache import InferenceParams, RecurrentInferenceParams
 
@@ -161,7 +161,38 @@ class StreamDecoder(KernelOps, nn.Module):
             self._gemm(a, pk.w, out, M, pk.Np, pk.Kp, EPI_NONE, variant=2 if M <= 512 else self.gemm_variant)
         return out
 
-    # ---- mixers shared by several families ---------------------------------------------------------
+    # ---- row kernels and mixers shared by several families -----------------------------------------
+    def _sum_norm(self, x, branches, outs, rows, gather=None, col_scale=None):
+        """x += col_scale * sum of the branches (y, ldy, norm weight or None, scale); outs: [(buffer, weight)] normed copies of the new x."""
+        cfg = self.config
+        p = SumNormParams(x=x.data_ptr(), n_branches=len(branches), eps=cfg.eps, dtype=self._dt, rows=rows, D=cfg.width,
+                          gather=gather.data_ptr() if gather is not None else None, ldo=_round_up(cfg.width, 64),
+                          col_scale=col_scale.data_ptr() if col_scale is not None else None)
+        for b, (y, ldy, nw, scale) in enumerate(branches):
+            p.y[b], p.ldy[b], p.norm_w[b], p.scale[b] = y.data_ptr(), ldy, (nw.data_ptr() if nw is not None else None), scale
+        for n, (o, wt) in enumerate(outs):
+            p.out[n], p.w[n] = o.data_ptr(), wt.data_ptr()
+        esz = 4 if self._dt else 2
+        nbytes = rows * cfg.width * (8.0 + esz * (len(branches) + len(outs)))
+        self._record("sum_norm", nbytes, lambda: check(_lib.lib().evo_sum_norm(C.byref(p), self._stream()), "evo_sum_norm"))
+
+    def _glu(self, z_ptr, up_ptr, ld, out, ldo, rows, F, act, limit=0.0, slope=1.0, route=None, group=0, n_groups=0, tail_w=0):
+        """out (rows, ldo) = act(gate) * up [* routing weight of the column's expert] (see evo_glu_act)."""
+        p = GluActParams(gate=z_ptr, up=up_ptr, ld=ld, out=out.data_ptr(), ldo=ldo, rows=rows, F=F, act=act, dtype=self._dt, limit=limit, slope=slope)
+        if route is not None:
+            p.group_w, p.ldw, p.group, p.n_groups, p.tail_w = route.data_ptr(), route.shape[1], group, n_groups, tail_w
+        self._record("glu_act", 3.0 * out.element_size() * rows * F, lambda: check(_lib.lib().evo_glu_act_ex(C.byref(p), self._stream()), "evo_glu_act"))
+
+    def _moe_route(self, h, M, router_w, E, top, correction=None, chosen=None, **kw):
+        """Routing weights (M, E + n_extra) fp32 from rows h (M, Kp); kw: further fields of evo_moe_route_params."""
+        n_extra = kw.get("n_extra", 0)
+        route = torch.empty(M, E + n_extra, dtype=torch.float32, device=h.device)
+        rp = MoeRouteParams(h=h.data_ptr(), ldh=h.shape[1], router_w=router_w.data_ptr(), correction=correction.data_ptr() if correction is not None else None,
+                            weights=route.data_ptr(), ldw=E + n_extra, chosen=chosen.data_ptr() if chosen is not None else None,
+                            rows=M, D=self.config.width, E=E, top=top, dtype=self._dt, **kw)
+        self._record("moe_route", float(M) * self.config.width * h.element_size(), lambda: check(_lib.lib().evo_moe_route_ex(C.byref(rp), self._stream()), "evo_moe_route"))
+        return route
+
     def _conv(self, r, src_ptr, ld, weight, bias, channels, taps, B, L, rec, fresh):
         """SiLU(short convolution) of `channels` columns starting at src_ptr -> (B*L, channels); the carried inputs live in rec.fir_state_dict[r]."""
         dev = weight.device
@@ -211,9 +242,9 @@ class StreamDecoder(KernelOps, nn.Module):
         self._record("gated_delta", 4.0 * M * m.heads * m.dim * m.vdim, lambda: check(_lib.lib().evo_gated_delta_fwd(C.byref(gp), ptr(ws), nws, self._stream()), "evo_gated_delta_fwd"))
         return self._linear(out, pk["out"], M), pk["out"].Np
 
-    def _run_chosen_experts(self, h, M, chosen, experts, ff, E, top):
+    def _run_chosen_experts(self, h, M, chosen, experts, ff, E, top, **act):
         """Only the chosen experts of a mixture: the (token, choice) pairs of `chosen` (M, top) int32 are sorted by expert, and every
-        expert ([gate ; up] and down weights, packed, hidden size ff, SiLU-gated) runs on its slice of the gathered rows of h (M, Kp).
+        expert ([gate ; up] and down weights, packed, hidden size ff; act: form and constants of the gate, SiLU by default) runs on its slice of the gathered rows of h (M, Kp).
         Returns (ys, slot_of): the experts' outputs in sorted order and the slot of every pair, for evo_moe_combine.  The per-expert
         row counts come back to the host (one round trip), so this does not run inside a captured step."""
         dev, lib = h.device, _lib.lib()
@@ -240,8 +271,7 @@ class StreamDecoder(KernelOps, nn.Module):
             up, down = experts[e]
             z = self._linear(hs[lo:lo + ne], up, ne)
             a = torch.empty(ne, down.Kp, dtype=self.act_dtype, device=dev)
-            self._record("glu_act", 3.0 * esz * ne * ff, lambda: check(lib.evo_glu_act(
-                ptr(z), C.c_void_p(z.data_ptr() + ff * esz), up.Np, ptr(a), down.Kp, ne, ff, 1, None, 0, 0, 0, 0, self._dt, self._stream()), "evo_glu_act"))
+            self._glu(z.data_ptr(), z.data_ptr() + ff * esz, up.Np, a, down.Kp, ne, ff, **(act or {"act": 1}))
             self._linear(a, down, ne, out=ys[lo:lo + ne])
         return ys, slot_of
 

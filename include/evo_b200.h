@@ -409,6 +409,16 @@ int evo_branch_norm(const evo_branch_norm_params* p, void* stream);
  * and for the columns after the groups w = group_w[r * ldw + n_groups] if tail_w is set, else 1; columns [F, ldo) are zero. */
 int evo_glu_act(const void* gate, const void* up, int64_t ld, void* out, int64_t ldo, int64_t rows, int F, int act,
                 const float* group_w, int64_t ldw, int group, int n_groups, int tail_w, int dtype, void* stream);
+/* The same with parameters in a struct and one more form:
+ *   act 3: out = c sigmoid(slope c) * (clamp(up, -limit, limit) + 1) * w  with c = min(gate, limit). */
+typedef struct {
+  const void* gate; const void* up; int64_t ld;
+  void* out; int64_t ldo; int64_t rows; int F, act;
+  const float* group_w; int64_t ldw; int group, n_groups, tail_w;
+  int dtype; float limit, slope;
+} evo_glu_act_params;
+int evo_glu_act_ex(const evo_glu_act_params* p, void* stream);
+
 /* out (rows, V) fp32 = in * mul */
 int evo_scale_logits(const void* in, int64_t ldi, float* out, int64_t rows, int V, float mul, int dtype, void* stream);
 
@@ -495,7 +505,8 @@ int evo_moe_combine(const void* ys, int64_t ldy, const void* base, int64_t ldb, 
  * Same conventions: `dtype` 0 = bf16 activations, 1 = fp32; weights and parameter vectors bf16. ==== */
 
 /* Closes a layer of up to EVO_SUM_NORM_BRANCHES parallel branches and opens the next one, one pass per row of the fp32 stream x (rows, D):
- *   x <- x + sum_b scale[b] * (norm_w[b] ? y[b] / sqrt(mean(y[b]^2) + eps) * norm_w[b] : y[b])
+ *   x <- x + col_scale * sum_b scale[b] * (norm_w[b] ? y[b] / sqrt(mean(y[b]^2) + eps) * norm_w[b] : y[b])
+ * (col_scale (D) bf16: a factor per column, NULL: 1)
  *   out[n] = x / sqrt(mean(x^2) + eps) * w[n]      for the outputs that are given (n < 2), pad columns [D, ldo) zero.
  * gather (rows) int64: row i reads stream row gather[i] (the branches are then added for the outputs only; x is not written back). */
 #define EVO_SUM_NORM_BRANCHES 3
@@ -509,6 +520,7 @@ typedef struct {
   int dtype;
   int64_t rows; int D;
   const int64_t* gather;
+  const void* col_scale;
 } evo_sum_norm_params;
 int evo_sum_norm(const evo_sum_norm_params* p, void* stream);
 
@@ -628,6 +640,50 @@ typedef struct {
 } evo_mlstm_params;
 size_t evo_mlstm_workspace(const evo_mlstm_params* p);
 int evo_mlstm_fwd(const evo_mlstm_params* p, void* workspace, size_t workspace_bytes, void* stream);
+
+/* ==== designs whose attention heads exchange scores before the softmax, beside a gated linear recurrence with a decay per key channel
+ * (Gagotar).  Same conventions: `dtype` 0 = bf16 activations, 1 = fp32; weights and parameter vectors bf16. ==== */
+
+/* Softmax attention over a linear key/value cache whose heads' scores are mixed before the softmax, with a chunked causal mask:
+ *   a_g = scale * temp[g] * q_g . k_(g / (H/G)),   s_h = sum_g talk[h*H + g] a_g,   softmax of s_h,   out = (sum_j p_j v_j) * sigmoid(gate[h])
+ *   query row r of a sequence sits at position i = pos + r (pos = *pos_dev if given, else q_pos0) and sees key j iff j <= i and, with
+ *   chunk > 0, floor(j / chunk) = floor(i / chunk).
+ *   q: head h at columns h*dk of a row; k / v: key head g at columns g*dk / g*dv of cache row j; temp (H), talk (H, H) bf16 (NULL: ones / identity);
+ *   gate (NULL: none): one column per head in a row.  Scores, their mixture and the softmax are fp32.  Pad columns [H*dv, ldo) are zeroed.
+ *   max_keys: with pos_dev, the most positions a sequence can have (sizes the key ranges of the step); cuda_cores: skip the tensor-core kernel.
+ * workspace: evo_mixed_attn_workspace() bytes (0 unless a query's keys are spread over several CTAs). */
+typedef struct {
+  const void* q; int64_t q_tok_stride;
+  const void* k; const void* v; int64_t k_tok_stride, v_tok_stride, k_batch_stride, v_batch_stride;
+  const void* gate; int64_t gate_tok_stride;
+  const void* temp; const void* talk;
+  void* out; int64_t ldo; int dtype;
+  int B; int64_t Lq; int H, G, dk, dv;
+  int64_t q_pos0; const int64_t* pos_dev; int64_t max_keys;
+  int64_t chunk; float scale; int cuda_cores;
+} evo_mixed_attn_params;
+size_t evo_mixed_attn_workspace(const evo_mixed_attn_params* p);
+int evo_mixed_attn_fwd(const evo_mixed_attn_params* p, void* workspace, size_t workspace_bytes, void* stream);
+
+/* Decays of a recurrence from a low-rank projection, fp32:  alpha[row*channels + c] = sigmoid(sum_r a2[c*rank + r] u[row*ldu + r] + bias[c]) ^ inv_tau. */
+int evo_low_rank_decay(const void* u, int64_t ldu, const void* a2, const void* bias, float inv_tau, float* alpha, int64_t rows, int rank, int channels, int dtype,
+                       void* stream);
+
+/* Gated linear attention, per head h over q, k (H*dk) and v (H*dv) of a row with one decay per key channel, alpha (rows, H*dk) fp32:
+ *   S <- diag(alpha) S + k v^T;   o = S^T (q q_scale);   out = o / sqrt(mean_c o^2 + eps) * norm_w[c] * silu(gate[h*dv + c])
+ * state (B, H, dk, dv) fp32 (zero_start: starts at 0).  workspace: evo_gla_workspace() bytes (0 unless a head's value channels are spread
+ * over several CTAs). */
+typedef struct {
+  const void* q; const void* k; const void* v; int64_t ld;
+  const float* alpha; float q_scale;
+  const void* gate; int64_t ld_gate; const void* norm_w; float eps;
+  float* state; int zero_start;
+  void* out; int64_t ldo; int dtype;
+  int B; int64_t L; int H, dk, dv;
+} evo_gla_params;
+size_t evo_gla_workspace(const evo_gla_params* p);
+int evo_gla_fwd(const evo_gla_params* p, void* workspace, size_t workspace_bytes, void* stream);
+
 
 #ifdef __cplusplus
 }
