@@ -1,6 +1,6 @@
 """bench.py — nucleotides/sec of the Evo-1 7B forward on B200 (BASELINE.json metric).
 
-    python bench.py [--gpus N] [--steps K] [--warmup W] [--workload 8k|131k|1k|32k|gen|zaverax|movalorn|nelovik|gakupel] [--impl ours|reference]
+    python bench.py [--gpus N] [--steps K] [--warmup W] [--workload 8k|131k|1k|32k|gen|zaverax|movalorn|nelovik|gakupel|gagotar] [--impl ours|reference]
 
 Workload "8k" (default): evo-1-8k-base scoring forward, batch 8 x
 8192 nt of synthetic uniform ACGT (+BOS => L = 8193), bf16, random-init weights of the 7B
@@ -13,7 +13,7 @@ collective (weak scaling); "131k" runs the sequence-parallel forward instead.
 Workload "zaverax" (an option; the default workload and its JSON contract are unchanged): the Zaverax design beside StripedHyena at
 equal layer sizes, prefill and decode, with a per-kernel roofline breakdown (bench_arch).  Workload "movalorn": the same for the
 Movalorn design beside Zaverax, the closest family.  Workload "nelovik": the Nelovik design beside Zaverax likewise.  Workload "gakupel":
-the Gakupel design beside Nelovik.
+the Gakupel design beside Nelovik.  Workload "gagotar": the Gagotar design beside Gakupel.
 --impl reference: the reference's own CPU implementation of the path.  stripedhyena==0.2.2 is
 not installable offline, so this arm times the oracle restatement (kind "port") on the host
 cores, rank 0 only, on a bounded sample of the same workload.
@@ -683,6 +683,26 @@ def _gakupel_models(size, dev):
     return gk, nv
 
 
+def _gagotar_models(size, dev):
+    """A Gagotar model and a Gakupel model (the closest family: fp32 stream, attention beside a matrix-state recurrence, experts) of equal
+    width, depth and head count, random weights.  Gagotar: four layers, each attention with mixed head scores (heads of 128 / 128, a fourth
+    as many key heads, fully rotated, chunks of 1100 positions) beside gated linear attention with heads of 128 x 128, and 16 experts (4
+    chosen) whose chosen hidden width equals Gakupel's."""
+    from evo_b200.gagotar import Gagotar, GagotarConfig
+    gk, nv = _gakupel_models(size, dev)
+    del nv
+    s = ARCH_SIZES[size]
+    d, H = s["width"], s["heads"]
+    ff = (8 * d // 3 + 255) // 256 * 256
+    layer = {"type": "parallel",
+             "mixer": {"left": {"heads": H, "kv_heads": H // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1100},
+                                "rot": {"dims": 128, "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}},
+                       "right": {"heads": H, "dim": 128, "vdim": 128, "tau": 16.0}},
+             "mlp": {"kind": "moe", "expert": {"ff": ff // 4, "limit": 7.0}, "router": {"experts": 16, "top": 4}}}
+    gc = {"architecture": "Gagotar", "vocab": 512, "width": d, "norm": {"eps": 1e-5}, "layers": [layer] * 4}
+    return Gagotar(GagotarConfig.from_dict(gc)).init_random(0, device=dev), gk
+
+
 def bench_arch(args):
     """--workload zaverax: prefill and decode throughput of the Zaverax design beside StripedHyena at equal layer sizes (random
     weights, 4 layers each, one of them attention), with a per-kernel breakdown against the measured rooflines.  Inputs are larger
@@ -696,16 +716,16 @@ def bench_arch(args):
     fp32_lane_ops = 148 * 128 * peaks.get("sm_max_mhz", 1965.0) * 1e6        # CUDA-core fp32 instructions (lanes) per second at the maximum clock
     bound = {"gemm": ("flop/s", peaks["bf16_tflops"] * 1e12), "gemm_simt": ("flop/s", 2 * fp32_lane_ops), "attn": ("flop/s", peaks["bf16_tflops"] * 1e12),
              "window_attn": ("flop/s", peaks["bf16_tflops"] * 1e12), "hgrn2": ("fp32 lane-op/s", fp32_lane_ops),
-             "gated_delta": ("fp32 lane-op/s", fp32_lane_ops), "ssd": ("fp32 lane-op/s", fp32_lane_ops), "mlstm": ("fp32 lane-op/s", fp32_lane_ops)}
+             "gated_delta": ("fp32 lane-op/s", fp32_lane_ops), "ssd": ("fp32 lane-op/s", fp32_lane_ops), "mlstm": ("fp32 lane-op/s", fp32_lane_ops), "gla": ("fp32 lane-op/s", fp32_lane_ops), "mixed_attn": ("flop/s", peaks["bf16_tflops"] * 1e12)}
     family = args.workload
-    other = {"zaverax": "stripedhyena", "movalorn": "zaverax", "nelovik": "zaverax", "gakupel": "nelovik"}[family]
+    other = {"zaverax": "stripedhyena", "movalorn": "zaverax", "nelovik": "zaverax", "gakupel": "nelovik", "gagotar": "gakupel"}[family]
     bound.update({"mingru": ("B/s", peaks["hbm_gbs"] * 1e9), "latent_decode": ("B/s", peaks["hbm_gbs"] * 1e9)})
     out = {"workload": family, "metric": f"tokens/sec, prefill and decode, {family} beside {other} at equal sizes", "unit": "tok/s", "dtype": "bf16",
            "data": "synthetic", "steps": steps, "warmup": warmup, "peaks": peaks, "sizes": {}}
     launches = 0
     with ClockSampler(0) as clocks:
         for size, s in ARCH_SIZES.items():
-            zv, sh = {"zaverax": _arch_models, "movalorn": _movalorn_models, "nelovik": _nelovik_models, "gakupel": _gakupel_models}[family](size, dev)
+            zv, sh = {"zaverax": _arch_models, "movalorn": _movalorn_models, "nelovik": _nelovik_models, "gakupel": _gakupel_models, "gagotar": _gagotar_models}[family](size, dev)
             rec = {}
             for name, model in ((family, zv), (other, sh)):
                 B, L = s["prefill"]
@@ -780,14 +800,14 @@ def main():
     ap.add_argument("--steps", type=int, default=None)
     ap.add_argument("--warmup", type=int, default=None)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="8k", choices=list(WORKLOADS) + ["zaverax", "movalorn", "nelovik", "gakupel"])
+    ap.add_argument("--workload", default="8k", choices=list(WORKLOADS) + ["zaverax", "movalorn", "nelovik", "gakupel", "gagotar"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-sub", action="store_true", help="default workload only: skip the sp131k / gen sub-records")
     ap.add_argument("--no-gen", action="store_true", help="skip the cached-generation sub-record")
     ap.add_argument("--sub-steps", type=int, default=3, help="timed steps of the 131k sub-record")
     ap.add_argument("--gen-tokens", type=int, default=None, help="new tokens of the end-to-end generate() run (default: 4096 = BASELINE configs[3])")
     args = ap.parse_args()
-    if args.workload in ("zaverax", "movalorn", "nelovik", "gakupel"):
+    if args.workload in ("zaverax", "movalorn", "nelovik", "gakupel", "gagotar"):
         return bench_arch(args)
     wl = WORKLOADS[args.workload]
     if args.impl == "reference":

@@ -131,7 +131,9 @@ class Gagotar(StreamDecoder):
                              chunk=a.chunk, scale=a.scale, cuda_cores=self.mixed_attn_cuda_cores)
         nws = lib.evo_mixed_attn_workspace(C.byref(ap))
         ws = torch.empty(nws, dtype=torch.uint8, device=dev) if nws else None
-        span = min(off + (L + 1) / 2.0, (a.chunk + 1) / 2.0) if a.chunk > 0 else off + (L + 1) / 2.0      # keys per query on average
+        c = a.chunk if a.chunk > 0 else off + L
+        seen = lambda n: n // c * (c * (c + 1) / 2.0) + (n % c) * (n % c + 1) / 2.0          # keys that the first n positions see together
+        span = (seen(off + L) - seen(off)) / L
         self._record("mixed_attn", 2.0 * M * a.heads * span * (a.dim + a.vdim),
                      lambda: check(lib.evo_mixed_attn_fwd(C.byref(ap), ptr(ws), nws, self._stream()), "evo_mixed_attn_fwd"))
         return self._linear(out, pk["left_out"], M), pk["left_out"].Np

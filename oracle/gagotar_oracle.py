@@ -161,3 +161,77 @@ def forward(tokens: List[int], W: Dict[str, torch.Tensor], cfg: dict, dtype=torc
         if taps is not None:
             taps.append(x)
     return (rms(x, eps) * W["final.norm"]) @ W["head"].T
+
+
+def make_config(mlps=("moe", "moe"), width=64, vocab=97, eps=1e-5, heads=4, kv_heads=2, dim=16, vdim=12, scale=0.3, chunk=24,
+                rot_dims=8, rot_base=1000.0, scaling=(8.0, 1.0, 4.0, 64), lin_heads=2, lin_dim=12, lin_vdim=20, tau=8.0,
+                experts=6, top=2, expert_ff=24, limit=1.2) -> dict:
+    """A small configuration in the checkpoints' own keys; every layer gets the same sizes (tests change single entries)."""
+    out = []
+    for mlp in mlps:
+        left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale}
+        if chunk:
+            left["mask"] = {"size": chunk}
+        if rot_dims:
+            left["rot"] = {"base": rot_base, "dims": rot_dims}
+            if scaling:
+                left["rot"]["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+        m = {"left": left, "right": {"heads": lin_heads, "dim": lin_dim, "vdim": lin_vdim, "tau": tau}}
+        f = {"kind": "moe", "expert": {"ff": expert_ff, "limit": limit}, "router": {"experts": experts, "top": top}} if mlp == "moe" else None
+        out.append({"type": "parallel", "mixer": m, "mlp": f})
+    return {"architecture": "Gagotar", "layers": out, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def tensor_shapes(cfg: dict, rank: int = 5) -> Dict[str, tuple]:
+    """Checkpoint tensor name -> shape for a configuration; rank: of the decay projection (no entry of the configuration gives it)."""
+    d, V = cfg["width"], cfg["vocab"]
+    out = {"embed": (V, d)}
+    for i, layer in enumerate(cfg["layers"]):
+        p = f"l{i}."
+        a, s = layer["mixer"]["left"], layer["mixer"]["right"]
+        H, G, dk, dv = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+        l, r = p + "mix.left.", p + "mix.right."
+        out.update({p + "norm1": (d,), p + "ls1": (d,), l + "q": (H * dk, d), l + "q.b": (H * dk,), l + "k": (G * dk, d), l + "k.b": (G * dk,), l + "v": (G * dv, d),
+                    l + "v.b": (G * dv,), l + "q.norm": (H * dk,), l + "k.norm": (G * dk,), l + "talk": (H, H), l + "temp": (H,), l + "g": (H, d), l + "o": (d, H * dv), l + "out": (d,)})
+        H, dk, dv = s["heads"], s["dim"], s["vdim"]
+        out.update({r + "q": (H * dk, d), r + "k": (H * dk, d), r + "v": (H * dv, d), r + "g": (H * dv, d), r + "o": (d, H * dv), r + "norm": (dv,),
+                    r + "a1": (rank, d), r + "a2": (H * dk, rank), r + "a2.b": (H * dk,), r + "out": (d,)})
+        f = layer.get("mlp")
+        if f is not None:
+            e = f["expert"]["ff"]
+            out.update({p + "norm2": (d,), p + "ls2": (d,), p + "mlp.router": (f["router"]["experts"], d)})
+            for k in range(f["router"]["experts"]):
+                out.update({f"{p}mlp.e{k}.gate": (e, d), f"{p}mlp.e{k}.up": (e, d), f"{p}mlp.e{k}.down": (d, e)})
+    out["final.norm"] = (d,)
+    out["head"] = (V, d)
+    return out
+
+
+def random_weights(cfg: dict, seed: int = 0, rank: int = 5) -> Dict[str, torch.Tensor]:
+    """Random bf16-representable weights of a usable scale."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in tensor_shapes(cfg, rank).items():
+        leaf = name.split(".")[-1]
+        if leaf in ("norm1", "norm2", "norm", "out"):
+            v = 1.0 + torch.randn(shape, generator=g) * 0.1
+        elif name.endswith("a2.b"):
+            v = torch.randn(shape, generator=g)
+        elif leaf == "b":
+            v = torch.randn(shape, generator=g) * 0.3
+        elif leaf in ("ls1", "ls2"):
+            v = 0.5 + torch.rand(shape, generator=g)
+        elif leaf == "temp":
+            v = 0.6 + 0.8 * torch.rand(shape, generator=g)
+        elif leaf == "talk":
+            v = torch.eye(shape[0]) + torch.randn(shape, generator=g) * 0.5
+        elif name == "embed":
+            v = torch.randn(shape, generator=g)
+        elif leaf in ("gate", "up"):
+            v = torch.randn(shape, generator=g) * 1.5 / math.sqrt(shape[-1])          # the limits are reached
+        elif leaf in ("a1", "a2"):
+            v = torch.randn(shape, generator=g) * 1.5 / math.sqrt(shape[-1])
+        else:
+            v = torch.randn(shape, generator=g) / math.sqrt(shape[-1])
+        out[name] = v.to(torch.bfloat16)
+    return out

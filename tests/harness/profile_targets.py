@@ -134,4 +134,27 @@ elif what in ("gakupel", "gakupel_step"):
             d["mha"].seqlen_offset = d["hyena"].seqlen_offset = ctx + t
             lg, _ = model(nxt, inference_params_dict=d)
     torch.cuda.synchronize()
+elif what in ("gagotar", "gagotar_step"):
+    # a 1-layer Gagotar model (mixed-score attention beside gated linear attention, 16 experts) at width 2048: one prompt of 2 x 4096 tokens
+    # ("gagotar": every prompt kernel once per forward) or single-token steps of 16 sequences behind 2048 tokens
+    from evo_b200.gagotar import Gagotar, GagotarConfig
+    layer = {"type": "parallel",
+             "mixer": {"left": {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1100}, "rot": {"dims": 128, "base": 500000.0}},
+                       "right": {"heads": 16, "dim": 128, "vdim": 128, "tau": 16.0}},
+             "mlp": {"kind": "moe", "expert": {"ff": 1408, "limit": 7.0}, "router": {"experts": 16, "top": 4}}}
+    gc = {"architecture": "Gagotar", "vocab": 512, "width": 2048, "norm": {"eps": 1e-5}, "layers": [layer]}
+    model = Gagotar(GagotarConfig.from_dict(gc)).init_random(0, device=dev)
+    if what == "gagotar":
+        ids = torch.randint(0, 512, (2, 4096), device=dev)
+        for _ in range(2):
+            model(ids)
+    else:
+        B, ctx = 16, 2048
+        d = model.initialize_inference_params(max_seqlen=ctx + 64, max_batch_size=B)
+        lg, d = model(torch.randint(0, 512, (B, ctx), device=dev), inference_params_dict=d)
+        nxt = lg[:, -1].argmax(-1, keepdim=True)
+        for t in range(3):
+            d["mha"].seqlen_offset = d["hyena"].seqlen_offset = ctx + t
+            lg, _ = model(nxt, inference_params_dict=d)
+    torch.cuda.synchronize()
 print("done", what)
