@@ -298,6 +298,7 @@ SIGNATURES = {
     "evo_glu_act_ex": (C.c_int, [C.POINTER(GluActParams), C.c_void_p]),
     "evo_mixed_attn_workspace": (C.c_size_t, [C.POINTER(MixedAttnParams)]),
     "evo_mixed_attn_fwd": (C.c_int, [C.POINTER(MixedAttnParams), C.c_void_p, C.c_size_t, C.c_void_p]),
+    "evo_mixed_attn_lost_waits": (C.c_int, [C.POINTER(C.c_uint)]),
     "evo_low_rank_decay": (C.c_int, [C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_float, C.c_void_p, C.c_int64, C.c_int, C.c_int, C.c_int, C.c_void_p]),
     "evo_gla_workspace": (C.c_size_t, [C.POINTER(GlaParams)]),
     "evo_gla_fwd": (C.c_int, [C.POINTER(GlaParams), C.c_void_p, C.c_size_t, C.c_void_p]),

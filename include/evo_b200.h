@@ -664,6 +664,8 @@ typedef struct {
 } evo_mixed_attn_params;
 size_t evo_mixed_attn_workspace(const evo_mixed_attn_params* p);
 int evo_mixed_attn_fwd(const evo_mixed_attn_params* p, void* workspace, size_t workspace_bytes, void* stream);
+/* Waits for a copy that ran out inside the prompt kernel since the library was loaded (0 unless a result is wrong); synchronises the device. */
+int evo_mixed_attn_lost_waits(unsigned int* count);
 
 /* Decays of a recurrence from a low-rank projection, fp32:  alpha[row*channels + c] = sigmoid(sum_r a2[c*rank + r] u[row*ldu + r] + bias[c]) ^ inv_tau. */
 int evo_low_rank_decay(const void* u, int64_t ldu, const void* a2, const void* bias, float inv_tau, float* alpha, int64_t rows, int rank, int channels, int dtype,

@@ -89,7 +89,8 @@ def _run_attention(q, k, v, scale, temp, talk, chunk, pos0, gate, dtype, rows, c
 # heads, key heads, dk, dv, chunk, rows, first position: one head, odd sizes, more than 8 / 16 / 32 heads (one, two, three CTAs per tile), wide heads
 ATT_SHAPES = [(4, 2, 16, 12, 24, 100, 0), (1, 1, 8, 8, 0, 50, 7), (3, 1, 10, 9, 17, 90, 37), (12, 4, 32, 48, 50, 120, 11), (16, 16, 24, 16, 64, 70, 0),
               (20, 5, 16, 24, 33, 70, 40), (33, 11, 8, 16, 40, 60, 25), (32, 8, 128, 128, 96, 130, 90), (16, 4, 128, 128, 0, 150, 100), (2, 2, 136, 136, 30, 40, 3),
-              (5, 5, 40, 72, 1, 20, 5), (17, 1, 20, 6, 28, 40, 0)]
+              (5, 5, 40, 72, 1, 20, 5), (17, 1, 20, 6, 28, 40, 0), (40, 8, 16, 120, 45, 50, 20),
+              (24, 6, 64, 64, 70, 80, 30), (3, 1, 192, 64, 37, 90, 13), (16, 16, 128, 128, 61, 50, 9), (6, 3, 72, 24, 100, 60, 150)]
 
 
 @pytest.mark.parametrize("H,G,dk,dv,chunk,L,pos0", ATT_SHAPES, ids=lambda v: str(v))
@@ -109,6 +110,34 @@ def test_mixed_attention_kernels_match_fp64(H, G, dk, dv, chunk, L, pos0):
     _close(_run_attention(*args, F32, L), want, 3e-5, "prompt rows, fp32")
     _close(_run_attention(*args, F32, 2), want, 3e-5, "two rows a call, fp32")
     _close(_run_attention(*args, B16, 1, device_pos=True), want, 1.2e-2, "steps with the position in device memory, bf16")
+
+
+@pytest.mark.parametrize("H,G,dk,dv", [(4, 2, 64, 64), (18, 6, 64, 128), (6, 3, 24, 40)])
+def test_mixed_attention_of_several_sequences_in_one_call(H, G, dk, dv):
+    """Each sequence has its own cache rows (whole column tiles through tensor maps, padded heads row by row); rows behind the last position hold NaNs."""
+    g = torch.Generator().manual_seed(dk)
+    B, L, pos0, rows, chunk = 3, 40, 21, 80, 33
+    q, kv = _bf(torch.randn(B, L, H * dk, generator=g)), torch.full((B, rows, G * (dk + dv)), float("nan"))
+    kv[:, :pos0 + L] = torch.randn(B, pos0 + L, G * (dk + dv), generator=g)
+    kv = _bf(kv)
+    talk = _bf(torch.eye(H) + torch.randn(H, H, generator=g) / math.sqrt(H))
+    qd, kvd, td = q.to(DEV), kv.to(DEV), talk.to(DEV)
+    cw, ldo = G * (dk + dv), (H * dv + 63) // 64 * 64
+    out = torch.full((B * L, ldo), 5.0, dtype=B16, device=DEV)
+    p = MixedAttnParams(q=qd.data_ptr(), q_tok_stride=H * dk, k=kvd.data_ptr(), v=kvd.data_ptr() + 2 * G * dk, k_tok_stride=cw, v_tok_stride=cw, k_batch_stride=rows * cw,
+                        v_batch_stride=rows * cw, talk=td.data_ptr(), out=out.data_ptr(), ldo=ldo, dtype=0, B=B, Lq=L, H=H, G=G, dk=dk, dv=dv, q_pos0=pos0, max_keys=rows,
+                        chunk=chunk, scale=0.9 / math.sqrt(dk))
+    lib = _lib.lib()
+    nws = lib.evo_mixed_attn_workspace(C.byref(p))
+    ws = torch.empty(max(nws, 1), dtype=torch.uint8, device=DEV)
+    check(lib.evo_mixed_attn_fwd(C.byref(p), ptr(ws), nws, _stream()))
+    for b in range(B):
+        k, v = kv[b, :pos0 + L, :G * dk].double().view(-1, G, dk), kv[b, :pos0 + L, G * dk:].double().view(-1, G, dv)
+        want = O.mixed_head_attention(q[b].double().view(L, H, dk), k, v, 0.9 / math.sqrt(dk), torch.ones(H, dtype=F64), talk.double(), chunk, pos0).reshape(L, H * dv)
+        _close(out[b * L:(b + 1) * L, :H * dv], want, 1.2e-2, f"sequence {b}")
+    lost = C.c_uint(99)
+    check(lib.evo_mixed_attn_lost_waits(C.byref(lost)))
+    assert lost.value == 0
 
 
 def test_mixed_attention_without_gate_temperature_and_mixture_is_plain_attention():
