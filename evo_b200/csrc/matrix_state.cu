@@ -10,8 +10,8 @@
 // every (key, query) pair read from shared memory then serves two columns, and the shared-memory pipe -- which bounded the
 // one-column form at half its time -- sees half the traffic per multiply-add.  Column j of the state belongs to LPC adjacent lanes of one warp, each
 // holding RPT rows in pairs (lane l, pair r: rows 2*(r*LPC + l) and + 1, so that the lanes of a column read consecutive 16-byte
-// (key, query, key, query) entries of shared memory, without bank conflicts); column sums (S^T k, S^T q) are folded with shuffles, so the time loop has no
-// barrier.  Value channels are independent in both recurrences: a head whose state does not fit one CTA's registers, or a call
+// (key, query, key, query) entries of shared memory, without bank conflicts); column sums (S^T k, S^T q) are folded with shuffles -- of four tokens together where the read-out does not feed the
+// state -- so the time loop has no barrier.  Value channels are independent in both recurrences: a head whose state does not fit one CTA's registers, or a call
 // that would leave SMs idle, is spread over several CTAs by value channel; the delta rule's read-outs then go to an fp32
 // workspace and a second small kernel applies the head norm, weight and gate.
 // Prompts on so few (head, sequence) pairs that every CTA has an SM of its own put 16 lanes with half the rows on a column of 65 to 128 rows
@@ -225,13 +225,13 @@ __global__ void __launch_bounds__(RPT <= 4 ? 1024 : (RPT <= 32 ? 512 : 256), 1) 
       }
     }
     // ---- time loop
-    for (int tt = 0; tt < nt; ++tt) {
-      float v[CPT];
+    if (MODE == MODE_DELTA) {
+      for (int tt = 0; tt < nt; ++tt) {
+        float v[CPT];
 #pragma unroll
-      for (int c = 0; c < CPT; ++c) v[c] = vs[tt * dvp + jl + c];
-      const float dec = MODE == MODE_GLA ? 0.f : sc[tt * 4 + 0];
-      const float4* e = reinterpret_cast<const float4*>(kq + tt * dkp) + l;             // two state rows per 16-byte read; pair r at e[r * LPC]
-      if (MODE == MODE_DELTA) {
+        for (int c = 0; c < CPT; ++c) v[c] = vs[tt * dvp + jl + c];
+        const float dec = sc[tt * 4 + 0];
+        const float4* e = reinterpret_cast<const float4*>(kq + tt * dkp) + l;           // two state rows per 16-byte read; pair r at e[r * LPC]
         constexpr bool KEEP = RPT <= 16;                   // the keys stay in registers for the update, or are read again
         float pk[CPT], pq[CPT], kx[KEEP ? RPT : 2];
 #pragma unroll
@@ -271,41 +271,71 @@ __global__ void __launch_bounds__(RPT <= 4 ? 1024 : (RPT <= 32 ? 512 : 256), 1) 
             else os[tt * dvp + jl + c] = o;
           }
         }
-      } else {
-        float y[CPT];
+      }
+    } else {
+      // TB tokens at a time: no token's read-out feeds the state, so their partial sums are folded over the column's lanes together -- each step
+      // halves the sums a lane still carries, NV - 1 shuffles and a few more instead of log2(LPC) per sum -- while the next tokens' products go on
+      constexpr int TB = 4, NV = TB * CPT;
+      for (int tb = 0; tb < nt; tb += TB) {
+        float y[NV];
 #pragma unroll
-        for (int c = 0; c < CPT; ++c) y[c] = 0.f;
-        if (MODE == MODE_MLSTM) {
-          const float inn = sc[tt * 4 + 1];
+        for (int u = 0; u < TB; ++u) {
 #pragma unroll
-          for (int c = 0; c < CPT; ++c) v[c] *= inn;
-        }
+          for (int c = 0; c < CPT; ++c) y[u * CPT + c] = 0.f;
+          const int tt = tb + u;
+          if (tt < nt) {
+            float v[CPT];
 #pragma unroll
-        for (int r = 0; r < RPT / 2; ++r) {
-          const float4 f = e[r * LPC];
-          const float2 d2 = MODE == MODE_GLA ? reinterpret_cast<const float2*>(al + tt * dkp)[r * LPC + l] : make_float2(dec, dec);
+            for (int c = 0; c < CPT; ++c) v[c] = vs[tt * dvp + jl + c];
+            const float dec = MODE == MODE_GLA ? 0.f : sc[tt * 4 + 0];
+            const float4* e = reinterpret_cast<const float4*>(kq + tt * dkp) + l;
+            if (MODE == MODE_MLSTM) {
+              const float inn = sc[tt * 4 + 1];
 #pragma unroll
-          for (int c = 0; c < CPT; ++c) {
-            S[c][2 * r] = fmaf(d2.x, S[c][2 * r], f.x * v[c]);          y[c] = fmaf(S[c][2 * r], f.y, y[c]);
-            S[c][2 * r + 1] = fmaf(d2.y, S[c][2 * r + 1], f.z * v[c]);  y[c] = fmaf(S[c][2 * r + 1], f.w, y[c]);
+              for (int c = 0; c < CPT; ++c) v[c] *= inn;
+            }
+#pragma unroll
+            for (int r = 0; r < RPT / 2; ++r) {
+              const float4 f = e[r * LPC];
+              const float2 d2 = MODE == MODE_GLA ? reinterpret_cast<const float2*>(al + tt * dkp)[r * LPC + l] : make_float2(dec, dec);
+#pragma unroll
+              for (int c = 0; c < CPT; ++c) {
+                S[c][2 * r] = fmaf(d2.x, S[c][2 * r], f.x * v[c]);          y[u * CPT + c] = fmaf(S[c][2 * r], f.y, y[u * CPT + c]);
+                S[c][2 * r + 1] = fmaf(d2.y, S[c][2 * r + 1], f.z * v[c]);  y[u * CPT + c] = fmaf(S[c][2 * r + 1], f.w, y[u * CPT + c]);
+              }
+            }
           }
         }
+        // after the fold lane l carries sums [first, first + left) of the column's NV (lanes beyond the NV-th repeat them)
+        int first = 0;
 #pragma unroll
-        for (int o = 1; o < LPC; o <<= 1)
+        for (int o = 1, n = NV; o < LPC; o <<= 1) {
+          if (n > 1) {
+            n >>= 1;
+            const bool up = l & o;
+            if (up) first += n;
 #pragma unroll
-          for (int c = 0; c < CPT; ++c) y[c] += __shfl_xor_sync(0xffffffffu, y[c], o);
-        if (MODE == MODE_MLSTM || MODE == MODE_GLA) {
-#pragma unroll
-          for (int c = 0; c < CPT; ++c)
-            if (l == 0) {
-              if (p.y) { if (j + c < dv) p.y[((row0 + tt) * p.H + h) * dv + j + c] = y[c]; }
-              else os[tt * dvp + jl + c] = y[c];
+            for (int q = 0; q < n; ++q) {
+              const float give = up ? y[q] : y[q + n], keep = up ? y[q + n] : y[q];
+              y[q] = keep + __shfl_xor_sync(0xffffffffu, give, o);
             }
-        } else {
-          const float Dv = sc[tt * 4 + 1];
+          } else {
+            y[0] += __shfl_xor_sync(0xffffffffu, y[0], o);
+          }
+        }
+        constexpr int LEFT = NV / LPC > 1 ? NV / LPC : 1;
 #pragma unroll
-          for (int c = 0; c < CPT; ++c)
-            if (l == 0 && j + c < dv) p.y[((row0 + tt) * p.H + h) * dv + j + c] = fmaf(Dv, v[c], y[c]);
+        for (int q = 0; q < LEFT; ++q) {
+          const int tt = tb + (first + q) / CPT, c = (first + q) % CPT;
+          if (l < NV && tt < nt) {
+            if (MODE == MODE_SSD) {
+              if (j + c < dv) p.y[((row0 + tt) * p.H + h) * dv + j + c] = fmaf(sc[tt * 4 + 1], vs[tt * dvp + jl + c], y[q]);
+            } else if (p.y) {
+              if (j + c < dv) p.y[((row0 + tt) * p.H + h) * dv + j + c] = y[q];
+            } else {
+              os[tt * dvp + jl + c] = y[q];
+            }
+          }
         }
       }
     }
