@@ -451,146 +451,146 @@ __global__ void __launch_bounds__(MAXH * 32) mixed_attn_mma_kernel(evo_mixed_att
     float* const Sn = Ss + (next & 1) * sbuf;                          // and of tile next
     const int vbuf = sh.nvb == 2 ? (next - 1) & 1 : 0;
     if (next > 0) {
-    // K of this tile and V of the previous one are no longer read
-    if (sh.vec) {
-      if (sh.nvb == 1 && next > 1) fetch(&vmap, vb, p.v_tok_stride, Vs, sh.vst, dv, DVP, k0, bar + 3);
-      if (more) fetch(&kmap, kb, p.k_tok_stride, Ks, sh.kst, dk, sh.dkp, k0 + KT, bar);
-      if (sh.nvb == 2) { if (more) fetch(&vmap, vb, p.v_tok_stride, Vs + (next & 1) * KT * sh.vst, sh.vst, dv, DVP, k0 + KT, bar + 3 + (next & 1)); }
-    } else {
-      fetch(&vmap, vb, p.v_tok_stride, Vs, sh.vst, dv, DVP, k0, bar);
-      if (more) fetch(&kmap, kb, p.k_tok_stride, Ks, sh.kst, dk, sh.dkp, k0 + KT, bar);
-    }
-    // ---- mixture: a warp takes every nw-th run of eight neighbouring places, four runs at a time
-    for (int nt0 = w; nt0 < QROWS * KT / 8; nt0 += 4 * nw) {
-      float D[4][4] = {};
-      uint32_t s[4];
-#pragma unroll
-      for (uint32_t u = 0; u < 4; ++u) {
-        const uint32_t nt = min((uint32_t)nt0 + u * nw, QROWS * KT / 8 - 1u);          // past the end: computed, not stored
-        s[u] = nt / (KT / 8) * SST + nt % (KT / 8) * 8;
+      // K of this tile and V of the previous one are no longer read
+      if (sh.vec) {
+        if (sh.nvb == 1 && next > 1) fetch(&vmap, vb, p.v_tok_stride, Vs, sh.vst, dv, DVP, k0, bar + 3);
+        if (more) fetch(&kmap, kb, p.k_tok_stride, Ks, sh.kst, dk, sh.dkp, k0 + KT, bar);
+        if (sh.nvb == 2) { if (more) fetch(&vmap, vb, p.v_tok_stride, Vs + (next & 1) * KT * sh.vst, sh.vst, dv, DVP, k0 + KT, bar + 3 + (next & 1)); }
+      } else {
+        fetch(&vmap, vb, p.v_tok_stride, Vs, sh.vst, dv, DVP, k0, bar);
+        if (more) fetch(&kmap, kb, p.k_tok_stride, Ks, sh.kst, dk, sh.dkp, k0 + KT, bar);
       }
-      const float* ta = Ts + qr * sh.tst + (lane & 3);
-      for (int ks = 0; ks < sh.hk / 8; ++ks) {
-        uint32_t th[4], tl[4];
-        const float* t = ta + ks * 8;
-        const float* sk = Sj + (ks * 8 + (lane & 3)) * PLANE + qr;
-        th[0] = __float_as_uint(t[0]); th[1] = __float_as_uint(t[8 * sh.tst]); th[2] = __float_as_uint(t[4]); th[3] = __float_as_uint(t[8 * sh.tst + 4]);
-        t += MAXH * sh.tst;
-        tl[0] = __float_as_uint(t[0]); tl[1] = __float_as_uint(t[8 * sh.tst]); tl[2] = __float_as_uint(t[4]); tl[3] = __float_as_uint(t[8 * sh.tst + 4]);
+      // ---- mixture: a warp takes every nw-th run of eight neighbouring places, four runs at a time
+      for (int nt0 = w; nt0 < QROWS * KT / 8; nt0 += 4 * nw) {
+        float D[4][4] = {};
+        uint32_t s[4];
+#pragma unroll
+        for (uint32_t u = 0; u < 4; ++u) {
+          const uint32_t nt = min((uint32_t)nt0 + u * nw, QROWS * KT / 8 - 1u);          // past the end: computed, not stored
+          s[u] = nt / (KT / 8) * SST + nt % (KT / 8) * 8;
+        }
+        const float* ta = Ts + qr * sh.tst + (lane & 3);
+        for (int ks = 0; ks < sh.hk / 8; ++ks) {
+          uint32_t th[4], tl[4];
+          const float* t = ta + ks * 8;
+          const float* sk = Sj + (ks * 8 + (lane & 3)) * PLANE + qr;
+          th[0] = __float_as_uint(t[0]); th[1] = __float_as_uint(t[8 * sh.tst]); th[2] = __float_as_uint(t[4]); th[3] = __float_as_uint(t[8 * sh.tst + 4]);
+          t += MAXH * sh.tst;
+          tl[0] = __float_as_uint(t[0]); tl[1] = __float_as_uint(t[8 * sh.tst]); tl[2] = __float_as_uint(t[4]); tl[3] = __float_as_uint(t[8 * sh.tst + 4]);
+#pragma unroll
+          for (int u = 0; u < 4; ++u) {
+            uint32_t b0h, b0l, b1h, b1l;
+            split_tf32(sk[s[u]], b0h, b0l);
+            split_tf32(sk[s[u] + 4 * PLANE], b1h, b1l);
+            mma_tf32(D[u], tl, b0h, b1h);
+            mma_tf32(D[u], th, b0l, b1l);
+            mma_tf32(D[u], th, b0h, b1h);
+          }
+        }
+        __syncwarp();
+        if (CLUSTER) wait_bounded(bar + 2, (next - 1) & 1);              // the own slots have been read by everyone
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
-          uint32_t b0h, b0l, b1h, b1l;
-          split_tf32(sk[s[u]], b0h, b0l);
-          split_tf32(sk[s[u] + 4 * PLANE], b1h, b1l);
-          mma_tf32(D[u], tl, b0h, b1h);
-          mma_tf32(D[u], th, b0l, b1l);
-          mma_tf32(D[u], th, b0h, b1h);
+          if (nt0 + u * nw >= QROWS * KT / 8) break;
+          float* dst = Sj + (h0 + qr) * PLANE + qc + s[u];
+          if (qr < nh) *reinterpret_cast<float2*>(dst) = make_float2(D[u][0], D[u][1]);
+          if (qr + 8 < nh) *reinterpret_cast<float2*>(dst + 8 * PLANE) = make_float2(D[u][2], D[u][3]);
         }
       }
       __syncwarp();
-      if (CLUSTER) wait_bounded(bar + 2, (next - 1) & 1);              // the own slots have been read by everyone
-#pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        if (nt0 + u * nw >= QROWS * KT / 8) break;
-        float* dst = Sj + (h0 + qr) * PLANE + qc + s[u];
-        if (qr < nh) *reinterpret_cast<float2*>(dst) = make_float2(D[u][0], D[u][1]);
-        if (qr + 8 < nh) *reinterpret_cast<float2*>(dst + 8 * PLANE) = make_float2(D[u][2], D[u][3]);
-      }
-    }
-    __syncwarp();
-    if (CLUSTER) cluster_arrive();                                     // this CTA's foreign score slots may be written again
-    if (sh.vec) wait_bounded(bar + 3 + vbuf, sh.nvb == 2 ? ((next - 1) >> 1) & 1 : (next - 1) & 1);
-    __syncthreads();
+      if (CLUSTER) cluster_arrive();                                     // this CTA's foreign score slots may be written again
+      if (sh.vec) wait_bounded(bar + 3 + vbuf, sh.nvb == 2 ? ((next - 1) >> 1) & 1 : (next - 1) & 1);
+      __syncthreads();
     }
     // ---- with two score buffers half of the warps of every scheduler score the next tile first, so that the stages use different pipes at the same time
 #pragma unroll 1
     for (int stage = 0; stage < 2; ++stage) {
-    if (stage == (sh.nsb == 2 ? (w >> 2) & 1 : 0)) {
-    // ---- softmax of the warp's head and P.V
-    if (on && next > 0) {
-      const float* src = Sj + slot + qr * SST + qc;
-      const uint32_t va = vaddr + vbuf * (KT * sh.vst * 2);
-      float P[KT / 8][4];
-      float mx0 = -INFINITY, mx1 = -INFINITY;
+      if (stage == (sh.nsb == 2 ? (w >> 2) & 1 : 0)) {
+        // ---- softmax of the warp's head and P.V
+        if (on && next > 0) {
+          const float* src = Sj + slot + qr * SST + qc;
+          const uint32_t va = vaddr + vbuf * (KT * sh.vst * 2);
+          float P[KT / 8][4];
+          float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
-      for (int n = 0; n < KT / 8; ++n) {
-        const float2 u0 = *reinterpret_cast<const float2*>(src + n * 8), u1 = *reinterpret_cast<const float2*>(src + 8 * SST + n * 8);
-        P[n][0] = u0.x; P[n][1] = u0.y; P[n][2] = u1.x; P[n][3] = u1.y;
-      }
-      if (k0 + KT - 1 > v_all || k0 < f_all) {                         // some row does not see the whole tile
-#pragma unroll
-        for (int n = 0; n < KT / 8; ++n)
-#pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            const int kj = k0 + n * 8 + qc + (c & 1);
-            if (c < 2 ? (kj > v0 || kj < f0) : (kj > v1 || kj < f1)) P[n][c] = -INFINITY;
+          for (int n = 0; n < KT / 8; ++n) {
+            const float2 u0 = *reinterpret_cast<const float2*>(src + n * 8), u1 = *reinterpret_cast<const float2*>(src + 8 * SST + n * 8);
+            P[n][0] = u0.x; P[n][1] = u0.y; P[n][2] = u1.x; P[n][3] = u1.y;
           }
-      }
+          if (k0 + KT - 1 > v_all || k0 < f_all) {                         // some row does not see the whole tile
 #pragma unroll
-      for (int n = 0; n < KT / 8; ++n) { mx0 = fmaxf(mx0, fmaxf(P[n][0], P[n][1])); mx1 = fmaxf(mx1, fmaxf(P[n][2], P[n][3])); }
-      mx0 = quad_max(mx0); mx1 = quad_max(mx1);
-      // the reference of the exponentials follows the maximum only when that has moved by more than 2^8: weights stay below 2^8, and the
-      // accumulators are seldom rescaled
-      if (!__all_sync(0xffffffffu, mx0 <= mrun[0] + 8.f && mx1 <= mrun[1] + 8.f)) {
-        const float mn0 = fmaxf(mrun[0], mx0), mn1 = fmaxf(mrun[1], mx1);
-        const float c0 = mn0 == -INFINITY ? 1.f : ex2(mrun[0] - mn0), c1 = mn1 == -INFINITY ? 1.f : ex2(mrun[1] - mn1);
-        lrun[0] *= c0; lrun[1] *= c1;
-        mrun[0] = mn0; mrun[1] = mn1;
+            for (int n = 0; n < KT / 8; ++n)
 #pragma unroll
-        for (int n = 0; n < NV8; ++n) { O[n][0] *= c0; O[n][1] *= c0; O[n][2] *= c1; O[n][3] *= c1; }
-      }
-      const float r0 = mrun[0] == -INFINITY ? 0.f : mrun[0], r1 = mrun[1] == -INFINITY ? 0.f : mrun[1];      // a row that has seen no key yet
+              for (int c = 0; c < 4; ++c) {
+                const int kj = k0 + n * 8 + qc + (c & 1);
+                if (c < 2 ? (kj > v0 || kj < f0) : (kj > v1 || kj < f1)) P[n][c] = -INFINITY;
+              }
+          }
 #pragma unroll
-      for (int kk = 0; kk < KT / 16; ++kk) {
+          for (int n = 0; n < KT / 8; ++n) { mx0 = fmaxf(mx0, fmaxf(P[n][0], P[n][1])); mx1 = fmaxf(mx1, fmaxf(P[n][2], P[n][3])); }
+          mx0 = quad_max(mx0); mx1 = quad_max(mx1);
+          // the reference of the exponentials follows the maximum only when that has moved by more than 2^8: weights stay below 2^8, and the
+          // accumulators are seldom rescaled
+          if (!__all_sync(0xffffffffu, mx0 <= mrun[0] + 8.f && mx1 <= mrun[1] + 8.f)) {
+            const float mn0 = fmaxf(mrun[0], mx0), mn1 = fmaxf(mrun[1], mx1);
+            const float c0 = mn0 == -INFINITY ? 1.f : ex2(mrun[0] - mn0), c1 = mn1 == -INFINITY ? 1.f : ex2(mrun[1] - mn1);
+            lrun[0] *= c0; lrun[1] *= c1;
+            mrun[0] = mn0; mrun[1] = mn1;
 #pragma unroll
-        for (int n = 2 * kk; n < 2 * kk + 2; ++n) {
-          P[n][0] = ex2(P[n][0] - r0); P[n][1] = ex2(P[n][1] - r0); P[n][2] = ex2(P[n][2] - r1); P[n][3] = ex2(P[n][3] - r1);
-          lrun[0] += P[n][0] + P[n][1]; lrun[1] += P[n][2] + P[n][3];              // this thread's share, folded over its quad at the end
+            for (int n = 0; n < NV8; ++n) { O[n][0] *= c0; O[n][1] *= c0; O[n][2] *= c1; O[n][3] *= c1; }
+          }
+          const float r0 = mrun[0] == -INFINITY ? 0.f : mrun[0], r1 = mrun[1] == -INFINITY ? 0.f : mrun[1];      // a row that has seen no key yet
+#pragma unroll
+          for (int kk = 0; kk < KT / 16; ++kk) {
+#pragma unroll
+            for (int n = 2 * kk; n < 2 * kk + 2; ++n) {
+              P[n][0] = ex2(P[n][0] - r0); P[n][1] = ex2(P[n][1] - r0); P[n][2] = ex2(P[n][2] - r1); P[n][3] = ex2(P[n][3] - r1);
+              lrun[0] += P[n][0] + P[n][1]; lrun[1] += P[n][2] + P[n][3];              // this thread's share, folded over its quad at the end
+            }
+            uint32_t ah[4], al[4];
+            cut_pack(P[2 * kk][0], P[2 * kk][1], ah[0], al[0]);
+            cut_pack(P[2 * kk][2], P[2 * kk][3], ah[1], al[1]);
+            cut_pack(P[2 * kk + 1][0], P[2 * kk + 1][1], ah[2], al[2]);
+            cut_pack(P[2 * kk + 1][2], P[2 * kk + 1][3], ah[3], al[3]);
+#pragma unroll
+            for (int n = 0; n < NV8; n += 4) {                             // four independent sums between a high part's product and the remainder's
+              uint32_t bv[2][4];
+#pragma unroll
+              for (int x = 0; x < 2; ++x)
+                ldmatrix_x4_trans_at(bv[x], SW ? va + (n >> 3) * (KT * 128) + kk * 2048 + (vx ^ (((n + 2 * x) & 6) << 4)) : va + kk * 32 * sh.vst + (n + 2 * x) * 16);
+#pragma unroll
+              for (int x = 0; x < 2; ++x) { mma_bf16(O[n + 2 * x], ah, bv[x][0], bv[x][1]); mma_bf16(O[n + 2 * x + 1], ah, bv[x][2], bv[x][3]); }
+#pragma unroll
+              for (int x = 0; x < 2; ++x) { mma_bf16(O[n + 2 * x], al, bv[x][0], bv[x][1]); mma_bf16(O[n + 2 * x + 1], al, bv[x][2], bv[x][3]); }
+            }
+          }
         }
-        uint32_t ah[4], al[4];
-        cut_pack(P[2 * kk][0], P[2 * kk][1], ah[0], al[0]);
-        cut_pack(P[2 * kk][2], P[2 * kk][3], ah[1], al[1]);
-        cut_pack(P[2 * kk + 1][0], P[2 * kk + 1][1], ah[2], al[2]);
-        cut_pack(P[2 * kk + 1][2], P[2 * kk + 1][3], ah[3], al[3]);
+      } else if (more) {
+        if (sh.vec) wait_bounded(bar, next & 1);
+        // ---- scores of the warp's head -> own slot, and a copy to the other CTAs
+        if (on) {
+          float S[KT / 8][4];
 #pragma unroll
-        for (int n = 0; n < NV8; n += 4) {                             // four independent sums between a high part's product and the remainder's
-          uint32_t bv[2][4];
-#pragma unroll
-          for (int x = 0; x < 2; ++x)
-            ldmatrix_x4_trans_at(bv[x], SW ? va + (n >> 3) * (KT * 128) + kk * 2048 + (vx ^ (((n + 2 * x) & 6) << 4)) : va + kk * 32 * sh.vst + (n + 2 * x) * 16);
-#pragma unroll
-          for (int x = 0; x < 2; ++x) { mma_bf16(O[n + 2 * x], ah, bv[x][0], bv[x][1]); mma_bf16(O[n + 2 * x + 1], ah, bv[x][2], bv[x][3]); }
-#pragma unroll
-          for (int x = 0; x < 2; ++x) { mma_bf16(O[n + 2 * x], al, bv[x][0], bv[x][1]); mma_bf16(O[n + 2 * x + 1], al, bv[x][2], bv[x][3]); }
-        }
-      }
-    }
-    } else if (more) {
-    if (sh.vec) wait_bounded(bar, next & 1);
-    // ---- scores of the warp's head -> own slot, and a copy to the other CTAs
-    if (on) {
-      float S[KT / 8][4];
-#pragma unroll
-      for (int n = 0; n < KT / 8; ++n) S[n][0] = S[n][1] = S[n][2] = S[n][3] = 0.f;
+          for (int n = 0; n < KT / 8; ++n) S[n][0] = S[n][1] = S[n][2] = S[n][3] = 0.f;
 #pragma unroll 2
-      for (int ks = 0; ks < sh.dkp / 16; ++ks) {
-        uint32_t a[4];                                                 // rows 0-7 / 8-15 x features 0-7 / 8-15
-        ldmatrix_x4_at(a, qaddr + ks * 32);
-        uint32_t kf[KT / 16][4];
+          for (int ks = 0; ks < sh.dkp / 16; ++ks) {
+            uint32_t a[4];                                                 // rows 0-7 / 8-15 x features 0-7 / 8-15
+            ldmatrix_x4_at(a, qaddr + ks * 32);
+            uint32_t kf[KT / 16][4];
 #pragma unroll
-        for (int n = 0; n < KT / 16; ++n)
-          ldmatrix_x4_at(kf[n], SW ? kaddr + (ks >> 2) * (KT * 128) + n * 2048 + (kx ^ ((ks & 3) << 5)) : kaddr + n * 32 * sh.kst + ks * 32);
+            for (int n = 0; n < KT / 16; ++n)
+              ldmatrix_x4_at(kf[n], SW ? kaddr + (ks >> 2) * (KT * 128) + n * 2048 + (kx ^ ((ks & 3) << 5)) : kaddr + n * 32 * sh.kst + ks * 32);
 #pragma unroll
-        for (int n = 0; n < KT / 16; ++n) { mma_bf16(S[2 * n], a, kf[n][0], kf[n][1]); mma_bf16(S[2 * n + 1], a, kf[n][2], kf[n][3]); }
+            for (int n = 0; n < KT / 16; ++n) { mma_bf16(S[2 * n], a, kf[n][0], kf[n][1]); mma_bf16(S[2 * n + 1], a, kf[n][2], kf[n][3]); }
+          }
+          float* dst = Sn + slot + qr * SST + qc;
+#pragma unroll
+          for (int n = 0; n < KT / 8; ++n) {
+            *reinterpret_cast<float2*>(dst + n * 8) = make_float2(S[n][0], S[n][1]);
+            *reinterpret_cast<float2*>(dst + 8 * SST + n * 8) = make_float2(S[n][2], S[n][3]);
+          }
+        }
       }
-      float* dst = Sn + slot + qr * SST + qc;
-#pragma unroll
-      for (int n = 0; n < KT / 8; ++n) {
-        *reinterpret_cast<float2*>(dst + n * 8) = make_float2(S[n][0], S[n][1]);
-        *reinterpret_cast<float2*>(dst + 8 * SST + n * 8) = make_float2(S[n][2], S[n][3]);
-      }
-    }
-    }
     }
     if (!more) break;
     if (CLUSTER) {
