@@ -119,7 +119,9 @@ class LatentPrepParams(C.Structure):
                 ("norm_w", C.c_void_p), ("eps", C.c_float), ("freq", C.c_void_p),
                 ("cache", C.c_void_p), ("cache_row", C.c_int64), ("cache_batch_stride", C.c_int64), ("rank_pad", C.c_int),
                 ("B", C.c_int), ("L", C.c_int64), ("H", C.c_int), ("dim", C.c_int), ("rot", C.c_int), ("rank", C.c_int),
-                ("pos0", C.c_int64), ("pos_dev", C.c_void_p), ("dtype", C.c_int), ("rot_dims", C.c_int)]
+                ("pos0", C.c_int64), ("pos_dev", C.c_void_p), ("dtype", C.c_int), ("rot_dims", C.c_int),
+                ("rot_len", C.c_float), ("dq", C.c_void_p), ("ld_dq", C.c_int64), ("dq_norm_w", C.c_void_p), ("q_rank", C.c_int),
+                ("cq", C.c_void_p), ("ld_cq", C.c_int64)]
 
 
 class LatentDecodeParams(C.Structure):
@@ -128,7 +130,8 @@ class LatentDecodeParams(C.Structure):
                 ("uk", C.c_void_p), ("uv", C.c_void_p), ("gate", C.c_void_p), ("ld_gate", C.c_int64),
                 ("out", C.c_void_p), ("ldo", C.c_int64),
                 ("B", C.c_int), ("Lq", C.c_int64), ("H", C.c_int), ("dim", C.c_int), ("rot", C.c_int), ("rank", C.c_int), ("vdim", C.c_int),
-                ("pos0", C.c_int64), ("pos_dev", C.c_void_p), ("window", C.c_int64), ("scale", C.c_float), ("dtype", C.c_int), ("max_keys", C.c_int64)]
+                ("pos0", C.c_int64), ("pos_dev", C.c_void_p), ("window", C.c_int64), ("scale", C.c_float), ("dtype", C.c_int), ("max_keys", C.c_int64),
+                ("gate_per_channel", C.c_int)]
 
 
 SUM_NORM_BRANCHES = 3
@@ -221,6 +224,12 @@ class GlaParams(C.Structure):
                 ("B", C.c_int), ("L", C.c_int64), ("H", C.c_int), ("dk", C.c_int), ("dv", C.c_int)]
 
 
+class DecayScanParams(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("ld", C.c_int64), ("decay", C.c_void_p), ("act", C.c_int), ("q_scale", C.c_float),
+                ("state", C.c_void_p), ("zero_start", C.c_int), ("y", C.c_void_p), ("dtype", C.c_int),
+                ("B", C.c_int), ("L", C.c_int64), ("H", C.c_int), ("dk", C.c_int), ("dv", C.c_int), ("recurrent", C.c_int)]
+
+
 # name -> (restype, argtypes); every symbol include/evo_b200.h declares
 SIGNATURES = {
     "evo_last_error": (C.c_char_p, []),
@@ -302,6 +311,10 @@ SIGNATURES = {
     "evo_low_rank_decay": (C.c_int, [C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_float, C.c_void_p, C.c_int64, C.c_int, C.c_int, C.c_int, C.c_void_p]),
     "evo_gla_workspace": (C.c_size_t, [C.POINTER(GlaParams)]),
     "evo_gla_fwd": (C.c_int, [C.POINTER(GlaParams), C.c_void_p, C.c_size_t, C.c_void_p]),
+    "evo_embed_scaled_f32": (C.c_int, [C.c_void_p, C.c_int, C.c_void_p, C.c_void_p, C.c_int64, C.c_int, C.c_int, C.c_float, C.c_void_p]),
+    "evo_decay_scan_workspace": (C.c_size_t, [C.POINTER(DecayScanParams)]),
+    "evo_decay_scan_fwd": (C.c_int, [C.POINTER(DecayScanParams), C.c_void_p, C.c_size_t, C.c_void_p]),
+    "evo_norm_gate": (C.c_int, [C.c_void_p, C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_int64, C.c_int64, C.c_int, C.c_float, C.c_int, C.c_void_p]),
     "evo_moe_route": (C.c_int, [C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int64, C.c_int, C.c_int, C.c_int, C.c_float, C.c_int, C.c_void_p]),
 }
 

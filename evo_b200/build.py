@@ -16,7 +16,7 @@ SOURCES = ["api.cu", "elementwise.cu", "hyena.cu", "gemm_tcgen05.cu", "gemm_smal
            "rowops.cu", "hgrn2.cu", "window_attention.cu", "window_attention_mma.cu", "gemm_simt.cu",
            "mingru.cu", "latent_attention.cu", "moe.cu",
            "branch_ops.cu", "matrix_state.cu", "attention_prep.cu", "post_norm.cu",
-           "mixed_attention.cu"]
+           "mixed_attention.cu", "linear_attention.cu"]
 # comparators for the GPU tests (cuBLASLt GEMM, CUDA-core attention): a separate library, never loaded by the product
 TEST_SRC = os.path.join(HERE, "..", "tests", "support", "test_support.cu")
 TEST_LIB = os.path.join(HERE, "..", "tests", "support", "libevo_b200_test.so")

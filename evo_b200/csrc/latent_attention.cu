@@ -2,7 +2,9 @@
 // all heads share; only [latent | rotated key part] is cached.
 //
 //   evo_latent_prep         one CTA per token: turns the rotated part of every query head in place (interleaved pairs, fp32 angles
-//                           pos * freq[i]), RMS-norms the latent (fp32) and appends [latent | 0.. | turned key part] to the cache.
+//                           pos * freq[i], one table per row for all heads), RMS-norms the latent (fp32) and appends
+//                           [latent | 0.. | turned key part] to the cache; where the queries come out of a latent of their own, it
+//                           norms that one too.  Each of the three parts can be left out.
 //   evo_latent_attn_decode  few query rows (the decoding step, short portions): the absorbed form, ql = Uk_h^T q_a, scores straight
 //                           against the cached latents, streaming softmax, the weighted sum of latents, then o = Uv_h . sum -- the
 //                           window's keys and values are never expanded, and every intermediate is fp32.  Four launches: absorb
@@ -63,22 +65,43 @@ __device__ __forceinline__ float block_max(float v, float* red) {
 
 template <typename T>
 __global__ void __launch_bounds__(128) latent_prep_kernel(evo_latent_prep_params p) {
+  extern __shared__ float tab[];                            // the row's cosines, then its sines, shared by all heads
   __shared__ float red[32];
   const int64_t row = blockIdx.x, b = row / p.L, t = row % p.L;
   const int64_t pos = (p.pos_dev ? (int64_t)*p.pos_dev : p.pos0) + t;
   const float fpos = (float)pos;
   const int half = p.rot_dims / 2, hd = p.dim + p.rot;      // entries [rot_dims, rot) of a rotated part pass unchanged
-  // queries: pair i of head h
-  T* q = (T*)p.q + row * p.ldq;
-  for (int idx = threadIdx.x; idx < p.H * half; idx += blockDim.x) {
-    const int h = idx / half, i = idx % half;
+  const float len = p.rot_len > 0.f ? p.rot_len : 1.f;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
     float s, c;
     sincosf(fpos * p.freq[i], &s, &c);
-    T* e = q + (int64_t)h * hd + p.dim + 2 * i;
-    const float u = ldf(e), v = ldf(e + 1);
-    stf(e, u * c - v * s);
-    stf(e + 1, v * c + u * s);
+    tab[i] = c * len;
+    tab[half + i] = s * len;
   }
+  __syncthreads();
+  // queries: pair i of head h
+  if (p.q) {
+    T* q = (T*)p.q + row * p.ldq;
+    for (int idx = threadIdx.x; idx < p.H * half; idx += blockDim.x) {
+      const int h = idx / half, i = idx % half;
+      const float c = tab[i], s = tab[half + i];
+      T* e = q + (int64_t)h * hd + p.dim + 2 * i;
+      const float u = ldf(e), v = ldf(e + 1);
+      stf(e, u * c - v * s);
+      stf(e + 1, v * c + u * s);
+    }
+  }
+  if (p.dq) {                                               // the queries' own latent, normed
+    const T* a = (const T*)p.dq + row * p.ld_dq;
+    T* o = (T*)p.cq + row * p.ld_cq;
+    const bf16* w = (const bf16*)p.dq_norm_w;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < p.q_rank; c += blockDim.x) { const float v = ldf(a + c); ss = fmaf(v, v, ss); }
+    ss = block_sum(ss, red);
+    const float rstd = 1.0f / sqrtf(ss / (float)p.q_rank + p.eps);
+    for (int c = threadIdx.x; c < p.ld_cq; c += blockDim.x) stf(o + c, c < p.q_rank ? ldf(a + c) * rstd * __bfloat162float(w[c]) : 0.f);
+  }
+  if (!p.dkv) return;
   const T* a = (const T*)p.dkv + row * p.ld_dkv;
   T* dst = (T*)p.cache + b * p.cache_batch_stride + pos * p.cache_row;
   float ss = 0.f;
@@ -88,8 +111,7 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(evo_latent_prep_params
   const bf16* w = (const bf16*)p.norm_w;
   for (int c = threadIdx.x; c < p.rank_pad; c += blockDim.x) stf(dst + c, c < p.rank ? ldf(a + c) * rstd * __bfloat162float(w[c]) : 0.f);
   for (int i = threadIdx.x; i < p.rot / 2; i += blockDim.x) {
-    float s = 0.f, c = 1.f;
-    if (i < half) sincosf(fpos * p.freq[i], &s, &c);
+    const float c = i < half ? tab[i] : 1.f, s = i < half ? tab[half + i] : 0.f;
     const float u = ldf(a + p.rank + 2 * i), v = ldf(a + p.rank + 2 * i + 1);
     stf(dst + p.rank_pad + 2 * i, u * c - v * s);
     stf(dst + p.rank_pad + 2 * i + 1, v * c + u * s);
@@ -181,15 +203,14 @@ __global__ void __launch_bounds__(DT) latent_decode_kernel(evo_latent_decode_par
     ql[r] = t * inv;                                                 // ql is free now: the normalised sum of latents
   }
   __syncthreads();
-  float gate = 1.f;
-  if (p.gate) gate = 1.f / (1.f + expf(-ldf((const T*)p.gate + row * p.ld_gate + h)));
+  const T* grow = p.gate ? (const T*)p.gate + row * p.ld_gate + (p.gate_per_channel ? (int64_t)h * p.vdim : h) : nullptr;
   const bf16* uv = (const bf16*)p.uv + (int64_t)h * p.vdim * rank;
   T* orow = (T*)p.out + row * p.ldo;
   for (int v = w; v < p.vdim; v += DT / 32) {
     float d = 0.f;
     for (int r = lane; r < rank; r += 32) d = fmaf(__bfloat162float(uv[(int64_t)v * rank + r]), ql[r], d);
     d = warp_sum(d);
-    if (lane == 0) stf(orow + (int64_t)h * p.vdim + v, d * gate);
+    if (lane == 0) stf(orow + (int64_t)h * p.vdim + v, grow ? d / (1.f + expf(-ldf(grow + (p.gate_per_channel ? v : 0)))) : d);
   }
   if (h == p.H - 1)
     for (int64_t c = (int64_t)p.H * p.vdim + tid; c < p.ldo; c += DT) stf(orow + c, 0.f);
@@ -570,7 +591,7 @@ __global__ void __launch_bounds__(256) latent_uv_kernel(evo_latent_decode_params
         for (int i = 0; i < nr; ++i) {
           const int64_t row = row0 + i;
           float gate = 1.f;
-          if (p.gate) gate = 1.f / (1.f + expf(-ldf((const T*)p.gate + row * p.ld_gate + h)));
+          if (p.gate) gate = 1.f / (1.f + expf(-ldf((const T*)p.gate + row * p.ld_gate + (p.gate_per_channel ? (int64_t)h * p.vdim + v : h))));
           stf((T*)p.out + row * p.ldo + (int64_t)h * p.vdim + v, d[i] * gate);
         }
     }
@@ -612,13 +633,17 @@ inline SplitPlan split_plan(const evo_latent_decode_params* p) {
 }  // namespace
 
 extern "C" int evo_latent_prep(const evo_latent_prep_params* p, void* stream) {
-  EVO_REQUIRE(p->q && p->dkv && p->norm_w && p->freq && p->cache, "evo_latent_prep: null argument");
-  EVO_REQUIRE(p->H > 0 && p->dim >= 0 && p->rot >= 0 && p->rot % 2 == 0 && p->rot_dims % 2 == 0 && p->rot_dims >= 0 && p->rot_dims <= p->rot && p->rank > 0 && p->rank_pad >= p->rank, "evo_latent_prep: bad shape");
-  EVO_REQUIRE(p->ldq >= (int64_t)p->H * (p->dim + p->rot) && p->ld_dkv >= p->rank + p->rot && p->cache_row >= p->rank_pad + p->rot, "evo_latent_prep: bad strides");
+  EVO_REQUIRE((p->q || p->dq || p->dkv) && (p->freq || p->rot_dims == 0), "evo_latent_prep: null argument");
+  EVO_REQUIRE(p->dim >= 0 && p->rot >= 0 && p->rot % 2 == 0 && p->rot_dims % 2 == 0 && p->rot_dims >= 0 && p->rot_dims <= p->rot, "evo_latent_prep: bad shape");
+  if (p->q) EVO_REQUIRE(p->H > 0 && p->ldq >= (int64_t)p->H * (p->dim + p->rot), "evo_latent_prep: bad query shape");
+  if (p->dq) EVO_REQUIRE(p->cq && p->dq_norm_w && p->q_rank > 0 && p->ld_dq >= p->q_rank && p->ld_cq >= p->q_rank, "evo_latent_prep: bad query latent");
+  if (p->dkv) EVO_REQUIRE(p->norm_w && p->cache && p->rank > 0 && p->rank_pad >= p->rank && p->ld_dkv >= p->rank + p->rot && p->cache_row >= p->rank_pad + p->rot, "evo_latent_prep: bad latent or cache row");
   if ((int64_t)p->B * p->L == 0) return 0;
   dim3 grid((unsigned)((int64_t)p->B * p->L)), block(128);
-  if (p->dtype) latent_prep_kernel<float><<<grid, block, 0, (cudaStream_t)stream>>>(*p);
-  else latent_prep_kernel<bf16><<<grid, block, 0, (cudaStream_t)stream>>>(*p);
+  const size_t smem = sizeof(float) * (size_t)p->rot_dims;
+  EVO_REQUIRE(smem <= 40 * 1024, "evo_latent_prep: too many rotated entries (%d)", p->rot_dims);
+  if (p->dtype) latent_prep_kernel<float><<<grid, block, smem, (cudaStream_t)stream>>>(*p);
+  else latent_prep_kernel<bf16><<<grid, block, smem, (cudaStream_t)stream>>>(*p);
   return check_launch("evo_latent_prep");
 }
 

@@ -2,6 +2,7 @@
 //   gated delta rule   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q        (evo_gated_delta_fwd)
 //   state-space dual   S <- a S + (dt B) x^T;  y = S^T C + D x                             (evo_ssd_fwd)
 //   per-channel decay  S <- diag(a) S + k v^T;  o = S^T q                                (evo_gla_fwd)
+//   constant decay     S <- a_h S + k v^T;  o = S^T q            (evo_decay_scan_fwd: fp32, steps and sizes without a block-wise form)
 //   matrix memory      m' = max(f + m, i);  S <- e^{f+m-m'} S + e^{i-m'} k v^T;  n alike;  o = S^T q / (max(|n.q|, e^{-m'}) + c)   (evo_mlstm_fwd)
 // with everything around them that the recurrence consumes computed here in fp32 from the activated projections: the unit norms of
 // q and k, sigmoid / softplus / exponentials of the per-head gates, and for the delta rule the head's RMS norm, weight and SiLU gate.
@@ -36,6 +37,10 @@
 
 using namespace evo;
 
+namespace evo {
+int decay_scan_recurrent(const evo_decay_scan_params* p, cudaStream_t st);      // called by linear_attention.cu
+}
+
 namespace {
 
 template <typename T> __device__ __forceinline__ float ldf(const T* p);
@@ -53,7 +58,7 @@ __device__ __forceinline__ float warp_sum(float v) {
 }
 
 constexpr int TCH = 16;      // tokens staged per round
-enum { MODE_DELTA = 0, MODE_SSD = 1, MODE_MLSTM = 2, MODE_GLA = 3 };
+enum { MODE_DELTA = 0, MODE_SSD = 1, MODE_MLSTM = 2, MODE_GLA = 3, MODE_CONST = 4 };
 
 // what both recurrences look like to the time loop
 struct ScanArgs {
@@ -70,12 +75,14 @@ struct ScanArgs {
   // matrix memory: gate biases, soft cap, running maximum (B, H), and beside y the reciprocal denominators per (row, head);
   // a head's state is its dk x dv matrix followed by the dk entries of the normaliser
   const void* i_bias; const void* f_bias; float cap, den_eps; float* mstate; float* em;
-  const float* alpha;                                              // per-channel decay: (rows, H*dk)
+  const float* alpha;                                              // per-channel decay: (rows, H*dk); constant decay: (H)
+  int act;                                                         // constant decay: 1 = keys, queries and values go through silu first
 };
 
 // soft cap c tanh(z / c) (c <= 0: none) and log sigmoid
 __device__ __forceinline__ float soft_cap(float z, float c) { return c > 0.f ? c * tanhf(z / c) : z; }
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float silu_if(float z, int act) { return act ? z / (1.f + expf(-z)) : z; }
 
 template <typename T, int RPT, int LPC, int MODE>
 __global__ void __launch_bounds__(RPT <= 4 ? 1024 : (RPT <= 32 ? 512 : 256), 1) matrix_state_kernel(ScanArgs p, int dvp) {
@@ -154,6 +161,13 @@ __global__ void __launch_bounds__(RPT <= 4 ? 1024 : (RPT <= 32 ? 512 : 256), 1) 
           sc[tt * 4 + 0] = log_sigmoid(soft_cap(gf, p.cap));
           sc[tt * 4 + 1] = soft_cap(gi, p.cap);
         }
+      } else if (MODE == MODE_CONST) {
+        for (int e = lane; e < dkp; e += 32) {
+          float2 o = make_float2(0.f, 0.f);
+          if (e < dk) { o.x = silu_if(ldf(kp + row * p.ld + e), p.act); o.y = silu_if(ldf(qp + row * p.ld + e), p.act) * p.q_scale; }
+          kq[tt * dkp + e] = o;
+        }
+        if (lane == 0) sc[tt * 4 + 0] = p.alpha[h];
       } else {
         const float dt = softplus_f(ldf((const T*)p.s0 + row * p.lds + h) + dtb);
         for (int e = lane; e < dkp; e += 32) {
@@ -163,7 +177,10 @@ __global__ void __launch_bounds__(RPT <= 4 ? 1024 : (RPT <= 32 ? 512 : 256), 1) 
         }
         if (lane == 0) { sc[tt * 4 + 0] = expf(-A * dt); sc[tt * 4 + 1] = Dh; }
       }
-      for (int c = lane; c < dvp; c += 32) vs[tt * dvp + c] = j0 + c < dv ? ldf(vp + row * p.ld + j0 + c) : 0.f;
+      for (int c = lane; c < dvp; c += 32) {
+        const float v = j0 + c < dv ? ldf(vp + row * p.ld + j0 + c) : 0.f;
+        vs[tt * dvp + c] = MODE == MODE_CONST ? silu_if(v, p.act) : v;
+      }
     }
     __syncthreads();
     if (MODE == MODE_MLSTM) {
@@ -474,7 +491,7 @@ int launch(const ScanArgs& a, const Plan& pl, cudaStream_t st, const char* what)
   if (smem > 48 * 1024) EVO_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   kern<<<dim3(a.H, a.B, pl.chunks), dim3(LPC * pl.dvc / columns_per_thread(RPT)), smem, st>>>(a, pl.dvc);
   int rc = check_launch(what);
-  if (rc || MODE == MODE_SSD || !a.y) return rc;
+  if (rc || MODE == MODE_SSD || MODE == MODE_CONST || !a.y) return rc;
   const int64_t warps = (int64_t)a.B * a.L * a.H;
   if (MODE == MODE_DELTA || MODE == MODE_GLA) delta_head_norm_kernel<T><<<(unsigned)((warps + 7) / 8), 256, 0, st>>>(a);
   else mlstm_head_norm_kernel<T><<<(unsigned)((warps + 7) / 8), 256, 0, st>>>(a);
@@ -485,7 +502,7 @@ template <typename T, int MODE>
 int dispatch(ScanArgs a, void* workspace, size_t workspace_bytes, cudaStream_t st, const char* what) {
   const Plan pl = plan(a.dk, a.dv, (int64_t)a.B * a.H, a.L);
   if (pl.rpt == 0) { set_error("%s: a state of %d rows per head does not fit (rows <= 2048)", what, a.dk); return -1; }
-  if (MODE != MODE_SSD && pl.chunks > 1) {
+  if (MODE != MODE_SSD && MODE != MODE_CONST && pl.chunks > 1) {
     const size_t rows = (size_t)a.B * a.L * a.H;
     const size_t need = sizeof(float) * rows * (a.dv + (MODE == MODE_MLSTM ? 1 : 0));
     if (!workspace || workspace_bytes < need) { set_error("%s: workspace too small (%zu < %zu)", what, workspace_bytes, need); return -1; }
@@ -643,4 +660,13 @@ extern "C" int evo_gla_fwd(const evo_gla_params* p, void* workspace, size_t work
   a.B = p->B; a.L = p->L; a.H = p->H; a.G = p->H; a.dk = p->dk; a.dv = p->dv;
   return p->dtype ? dispatch<float, MODE_GLA>(a, workspace, workspace_bytes, (cudaStream_t)stream, "evo_gla_fwd")
                   : dispatch<bf16, MODE_GLA>(a, workspace, workspace_bytes, (cudaStream_t)stream, "evo_gla_fwd");
+}
+
+// constant decay, token by token (linear_attention.cu holds the entry point and the block-wise form)
+int evo::decay_scan_recurrent(const evo_decay_scan_params* p, cudaStream_t st) {
+  ScanArgs a = {};
+  a.kk = p->k; a.qq = p->q; a.vv = p->v; a.ld = p->ld; a.alpha = p->decay; a.act = p->act; a.q_scale = p->q_scale;
+  a.state = p->state; a.zero_start = p->zero_start; a.y = p->y;
+  a.B = p->B; a.L = p->L; a.H = p->H; a.G = p->H; a.dk = p->dk; a.dv = p->dv;
+  return p->dtype ? dispatch<float, MODE_CONST>(a, nullptr, 0, st, "evo_decay_scan_fwd") : dispatch<bf16, MODE_CONST>(a, nullptr, 0, st, "evo_decay_scan_fwd");
 }

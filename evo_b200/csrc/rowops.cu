@@ -45,12 +45,12 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 // ------------------------------------------------------------------ embedding gather into the fp32 stream
 template <typename IdT>
 __global__ void embed_f32_kernel(const IdT* __restrict__ ids, const bf16* __restrict__ table, float* __restrict__ out,
-                                 int64_t n_tokens, int D, int vocab) {
+                                 int64_t n_tokens, int D, int vocab, float scale) {
   const int64_t row = blockIdx.x;
   long long id = (long long)ids[row];
   id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
   const bf16* src = table + (int64_t)id * D;
-  for (int c = threadIdx.x; c < D; c += blockDim.x) out[row * D + c] = __bfloat162float(src[c]);
+  for (int c = threadIdx.x; c < D; c += blockDim.x) out[row * D + c] = __bfloat162float(src[c]) * scale;
 }
 
 // ------------------------------------------------------------------ residual update + RMS norm
@@ -246,12 +246,16 @@ __global__ void copy_rows_kernel(const T* __restrict__ src, int64_t lds, T* __re
 
 }  // namespace
 
-extern "C" int evo_embed_f32(const void* ids, int ids_are_i64, const void* table, float* out, int64_t n_tokens, int D, int vocab, void* stream) {
+extern "C" int evo_embed_scaled_f32(const void* ids, int ids_are_i64, const void* table, float* out, int64_t n_tokens, int D, int vocab, float scale, void* stream) {
   if (n_tokens == 0) return 0;
   dim3 grid((unsigned)n_tokens), block(128);
-  if (ids_are_i64) embed_f32_kernel<long long><<<grid, block, 0, (cudaStream_t)stream>>>((const long long*)ids, (const bf16*)table, out, n_tokens, D, vocab);
-  else embed_f32_kernel<int><<<grid, block, 0, (cudaStream_t)stream>>>((const int*)ids, (const bf16*)table, out, n_tokens, D, vocab);
+  if (ids_are_i64) embed_f32_kernel<long long><<<grid, block, 0, (cudaStream_t)stream>>>((const long long*)ids, (const bf16*)table, out, n_tokens, D, vocab, scale);
+  else embed_f32_kernel<int><<<grid, block, 0, (cudaStream_t)stream>>>((const int*)ids, (const bf16*)table, out, n_tokens, D, vocab, scale);
   return check_launch("evo_embed_f32");
+}
+
+extern "C" int evo_embed_f32(const void* ids, int ids_are_i64, const void* table, float* out, int64_t n_tokens, int D, int vocab, void* stream) {
+  return evo_embed_scaled_f32(ids, ids_are_i64, table, out, n_tokens, D, vocab, 1.0f, stream);
 }
 
 extern "C" int evo_resid_norm(const evo_resid_norm_params* p, void* stream) {

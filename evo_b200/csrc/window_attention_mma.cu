@@ -8,7 +8,7 @@
 // strides are multiples of 8 -- asynchronous ones into two buffers, the next tile on its way while the current one is in work, as
 // long as two CTAs still fit an SM's shared memory.  A warp keeps both maps' output accumulators (16 x dv fp32 each) in registers and handles one map
 // at a time (scores -> softmax -> P.V), so only one 16 x 64 tile of probabilities is live.
-// Head sizes are padded to 16 in shared memory (zero columns); dk <= 128, dv <= 128 and dv % 8 == 0, otherwise the CUDA-core
+// Head sizes are padded to 16 in shared memory (zero columns); maps x dk <= 256, dv <= 128 and dv % 8 == 0, otherwise the CUDA-core
 // kernel runs.  The tile walk is the CUDA-core kernel's: [0, keep_first), the pooled blocks that the CTA's last query sees, and the
 // union of the CTA's windows.  A soft cap is applied to the fp32 scores before the softmax (tanh from ex2 and a division), and a
 // sink enters the denominators at the end; a distance bias is taken off the fp32 scores together with the mask.
@@ -355,6 +355,6 @@ int dispatch(const evo_window_attn_params* p, cudaStream_t st) {
 }  // namespace
 
 int evo::window_attn_mma(const evo_window_attn_params* p, cudaStream_t st) {
-  if (p->dtype != 0 || p->dk * p->n_maps > 256 || p->dk > 128 || p->dv > 128 || p->dv % 8 != 0 || p->Lq < 16) return 1;
+  if (p->dtype != 0 || p->dk * p->n_maps > 256 || p->dv > 128 || p->dv % 8 != 0 || p->Lq < 16) return 1;
   return p->n_maps == 2 ? dispatch<2>(p, st) : dispatch<1>(p, st);
 }

@@ -148,6 +148,13 @@ def _load_gagotar(model_dir: str, config: dict, device, dtype, **kwargs):
     return _load_flat(family, model_dir, config, device, dtype)
 
 
+def _load_nilatar(model_dir: str, config: dict, device, dtype, **kwargs):
+    def family():
+        from .nilatar import Nilatar, NilatarConfig
+        return Nilatar, NilatarConfig
+    return _load_flat(family, model_dir, config, device, dtype)
+
+
 def _load_stripedhyena(model_dir: str, config: dict, device, dtype, model_name: str = "evo-1-8k-base", **kwargs):
     if dtype not in (None, torch.bfloat16):
         raise NotImplementedError("StripedHyena runs in bfloat16 (fp32 poles and residues) only")
@@ -161,6 +168,7 @@ ARCHITECTURES = {
     "Nelovik": (_load_nelovik, (torch.bfloat16, torch.float32)),
     "Gakupel": (_load_gakupel, (torch.bfloat16, torch.float32)),
     "Gagotar": (_load_gagotar, (torch.bfloat16, torch.float32)),
+    "Nilatar": (_load_nilatar, (torch.bfloat16, torch.float32)),
     "StripedHyena": (_load_stripedhyena, (torch.bfloat16,)),
     "StripedHyenaModelForCausalLM": (_load_stripedhyena, (torch.bfloat16,)),
 }

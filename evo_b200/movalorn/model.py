@@ -27,13 +27,12 @@ from typing import Optional
 import torch
 
 from .. import _lib
-from .._lib import BranchNormParams, LatentDecodeParams, LatentPrepParams, MinGruParams, WindowAttnParams, check, ptr
+from .._lib import BranchNormParams, MinGruParams, check, ptr
 from ..stream_model import StreamDecoder, _Packed, _round_up
 from ..stripedhyena.cache import InferenceParams, RecurrentInferenceParams
 from .config import MovalornConfig
 
 PREV_TOKEN = -1               # key of the last-token vector in the recurrent state holder
-ABSORBED_MAX_ROWS = 4         # portions up to this many tokens attend straight from the latent cache
 
 
 class _Pending:
@@ -51,8 +50,6 @@ class Movalorn(StreamDecoder):
 
     def __init__(self, config: MovalornConfig, dtype: torch.dtype = torch.bfloat16):
         super().__init__(config, dtype)
-        # few-row latent attention: "shared" = heads share each tile of latents (three launches), "head" = one CTA per (query, head)
-        self.latent_decode_path = os.environ.get("EVO_B200_LATENT_DECODE", "shared")
         # expert mixtures: calls with at least this many rows (outside a captured step) run only the chosen experts, one GEMM pair per
         # expert over the rows sorted by expert (the per-expert row counts come back to the host); fewer rows run all experts densely
         self.moe_sparse_min_rows = int(os.environ.get("EVO_B200_MOE_SPARSE_MIN_ROWS", "1024"))
@@ -99,18 +96,7 @@ class Movalorn(StreamDecoder):
                 e["in"] = _Packed(torch.cat([w[p + "mix.z"], w[p + "mix.x"], w[p + "mix.g"], w[p + "rg1"]], 0))
             else:
                 e["in"] = _Packed(torch.cat([w[p + "mix.q"], w[p + "mix.dkv"], w[p + "mix.g"], w[p + "rg1"]], 0))
-                # expansion of cache rows [latent | 0.. | rotated key part] into per-head keys [Uk_h c | rotated part] and values Uv_h c:
-                # identity rows carry the shared rotated part into every head's key
-                rank_pad = _round_up(m.kv_rank, 8)
-                hd = m.dim + m.rot_dim
-                up = torch.zeros(m.heads * hd + m.heads * m.vdim, rank_pad + m.rot_dim, dtype=torch.bfloat16, device=dev)
-                for h in range(m.heads):
-                    up[h * hd:h * hd + m.dim, :m.kv_rank] = w[p + "mix.uk"][h * m.dim:(h + 1) * m.dim]
-                    up[h * hd + m.dim:(h + 1) * hd, rank_pad:] = torch.eye(m.rot_dim, dtype=torch.bfloat16, device=dev)
-                up[m.heads * hd:, :m.kv_rank] = w[p + "mix.uv"]
-                e["expand"] = _Packed(up)
-                e["rank_pad"] = rank_pad
-                e["cache_row"] = e["expand"].Kp
+                e["latent"] = self._pack_latent(m, w[p + "mix.uk"], w[p + "mix.uv"])
                 i2 = torch.arange(0, m.rot_dims, 2, dtype=torch.float32)
                 e["freq"] = (torch.tensor(m.rot_base, dtype=torch.float32) ** (-i2 / m.rot_dims)).to(dev) if m.rot_dims else torch.zeros(1, device=dev)
             e["out"] = _Packed(w[p + "mix.o"])
@@ -180,55 +166,14 @@ class Movalorn(StreamDecoder):
 
     def _latent_attention(self, r, i, m, h, B, L, ip: Optional[InferenceParams], off: int, pos_dev):
         pk = self._packed["layers"][i]
-        M, dev, w, lib = B * L, h.device, self.weights, _lib.lib()
+        M, w, p = B * L, self.weights, f"l{i}."
         z = self._linear(h, pk["in"], M)
         esz, ld = z.element_size(), pk["in"].Np
-        hd = m.dim + m.rot_dim
-        qw, aw = m.heads * hd, m.kv_rank + m.rot_dim
-        rank_pad, cache_row = pk["rank_pad"], pk["cache_row"]
-        if ip is None:
-            cache = torch.zeros(B, L, cache_row, dtype=self.act_dtype, device=dev)
-        else:
-            cache = self._kv_rows(ip, r, cache_row, B, off, L, pos_dev)
-        bstride = cache.shape[1] * cache_row
-        pos_ptr = pos_dev.data_ptr() if pos_dev is not None else None
-        pp = LatentPrepParams(q=z.data_ptr(), ldq=ld, dkv=z.data_ptr() + qw * esz, ld_dkv=ld, norm_w=w[f"l{i}.mix.dkv.norm"].data_ptr(), eps=self.config.eps,
-                              freq=pk["freq"].data_ptr(), cache=cache.data_ptr(), cache_row=cache_row, cache_batch_stride=bstride, rank_pad=rank_pad,
-                              B=B, L=L, H=m.heads, dim=m.dim, rot=m.rot_dim, rank=m.kv_rank, pos0=off, pos_dev=pos_ptr, dtype=self._dt, rot_dims=m.rot_dims)
-        self._record("latent_prep", float(M) * (qw + 2 * aw) * esz, lambda: check(lib.evo_latent_prep(C.byref(pp), self._stream()), "evo_latent_prep"))
-        inner = m.heads * m.vdim
-        ldo = _round_up(inner, 64)
-        out = torch.empty(M, ldo, dtype=self.act_dtype, device=dev)
-        gate_ptr = z.data_ptr() + (qw + aw) * esz
-        span = min(off + L, m.window) if m.window > 0 else off + (L + 1) / 2.0
-        if L <= ABSORBED_MAX_ROWS or pos_dev is not None:
-            dp = LatentDecodeParams(q=z.data_ptr(), ldq=ld, cache=cache.data_ptr(), cache_row=cache_row, cache_batch_stride=bstride, rank_pad=rank_pad,
-                                    uk=w[f"l{i}.mix.uk"].data_ptr(), uv=w[f"l{i}.mix.uv"].data_ptr(), gate=gate_ptr, ld_gate=ld,
-                                    out=out.data_ptr(), ldo=ldo, B=B, Lq=L, H=m.heads, dim=m.dim, rot=m.rot_dim, rank=m.kv_rank, vdim=m.vdim,
-                                    pos0=off, pos_dev=pos_ptr, window=m.window, scale=m.scale, dtype=self._dt,
-                                    max_keys=cache.shape[1] if pos_dev is not None else off + L)
-            nws = lib.evo_latent_attn_decode_workspace(C.byref(dp)) if self.latent_decode_path == "shared" else 0
-            ws = torch.empty(nws, dtype=torch.uint8, device=dev) if nws else None
-            # roofline bytes: each sequence's visible latents once (all heads share them)
-            self._record("latent_decode", float(M) * span * (m.kv_rank + m.rot_dim) * esz,
-                         lambda: check(lib.evo_latent_attn_decode(C.byref(dp), ptr(ws), nws, self._stream()), "evo_latent_attn_decode"))
-        else:
-            lo = max(0, off - (m.window - 1)) if m.window > 0 else 0
-            n = off + L - lo
-            ex = pk["expand"]
-            kv = torch.empty(B, n, ex.Np, dtype=self.act_dtype, device=dev)
-            for b in range(B):
-                self._linear(cache[b, lo:off + L], ex, n, out=kv[b])
-            ap = WindowAttnParams(q=z.data_ptr(), q_tok_stride=ld, gate=gate_ptr, gate_tok_stride=ld, gate_per_head=1,
-                                  k=kv.data_ptr() - lo * ex.Np * esz, v=kv.data_ptr() + (qw - lo * ex.Np) * esz,
-                                  k_tok_stride=ex.Np, v_tok_stride=ex.Np, k_batch_stride=n * ex.Np, v_batch_stride=n * ex.Np,
-                                  out=out.data_ptr(), ldo=ldo, dtype=self._dt, B=B, Lq=L, H=m.heads, G=m.heads, dk=hd, dv=m.vdim, n_maps=1,
-                                  q_pos0=off, pos_dev=None, window=m.window, keep_first=0, scale=m.scale, lambda_=0.0, head_norm=0,
-                                  norm_eps=self.config.eps, out_scale=1.0)
-            self._record("window_attn", 4.0 * M * m.heads * span * (hd + m.vdim),
-                         lambda: check(lib.evo_window_attn_fwd(C.byref(ap), self._stream()), "evo_window_attn_fwd"))
+        qw, aw = m.heads * (m.dim + m.rot_dim), m.kv_rank + m.rot_dim
+        cache = self._latent_rows(r, m, pk["latent"], z.data_ptr() + qw * esz, ld, w[p + "mix.dkv.norm"], pk["freq"], 1.0, B, L, ip, off, pos_dev, q=(z.data_ptr(), ld))
+        out = self._latent_attend(m, pk["latent"], z.data_ptr(), ld, cache, w[p + "mix.uk"], w[p + "mix.uv"], z.data_ptr() + (qw + aw) * esz, ld, False, B, L, off, pos_dev)
         y = self._linear(out, pk["out"], M)
-        return _Pending(y, pk["out"].Np, z.data_ptr() + (qw + aw + m.heads) * esz, ld, w[f"l{i}.rg1.b"], self._packed["gain"][f"l{i}.norm1b"], hold=z)
+        return _Pending(y, pk["out"].Np, z.data_ptr() + (qw + aw + m.heads) * esz, ld, w[p + "rg1.b"], self._packed["gain"][p + "norm1b"], hold=z)
 
     def _sparse_pack(self, i, f):
         pk = self._packed["layers"][i]

@@ -1,5 +1,5 @@
 """Shared base of the model families that keep the residual stream in fp32 and are described by a flat table of checkpoint
-tensors (Zaverax, Movalorn, Nelovik, Gakupel, Gagotar): weight holding and strict loading, the padded GEMM weights, the linear-layer dispatch
+tensors (Zaverax, Movalorn, Nelovik, Gakupel, Gagotar, Nilatar): weight holding and strict loading, the padded GEMM weights, the linear-layer dispatch
 (tcgen05 GEMMs for bf16 activations, the CUDA-core fp32 GEMM for the all-fp32 mode), the inference-state holders, the
 forward protocol and the on-device generation loop.  A family provides `_ensure_packed()` and
 `_body(ids, B, L, state, offset, pos_dev=None, rows=None) -> fp32 logits`; everything that drives a model -- the generation loop,
@@ -23,9 +23,13 @@ import torch
 import torch.nn as nn
 
 from . import _lib
-from ._lib import EPI_NONE, ConvActParams, GatedDeltaParams, GluActParams, MoeRouteParams, SumNormParams, check, ptr
+from ._lib import (EPI_NONE, ConvActParams, GatedDeltaParams, GluActParams, LatentDecodeParams, LatentPrepParams, MoeRouteParams, SumNormParams, WindowAttnParams,
+                   check, ptr)
 from .engine import KernelOps
 from .stripedhyena.cache import InferenceParams, RecurrentInferenceParams
+
+
+ABSORBED_MAX_ROWS = 4         # latent attention: portions up to this many tokens attend straight from the latent cache
 
 
 def _round_up(x: int, m: int) -> int:
@@ -61,6 +65,8 @@ class StreamDecoder(KernelOps, nn.Module):
         self.gemm_path = os.environ.get(self.gemm_env, "tc")
         self.gemm_variant = int(os.environ.get("EVO_B200_GEMM_VARIANT", "0"))
         self.gemm_variant_gate = self.gemm_variant
+        # few-row latent attention: "shared" = heads share each tile of latents (three launches), "head" = one CTA per (query, head)
+        self.latent_decode_path = os.environ.get("EVO_B200_LATENT_DECODE", "shared")
         self.decode_graph = os.environ.get("EVO_B200_DECODE_GRAPH", "1") != "0"
         self._smallm_ws = None
         self._decode = None
@@ -241,6 +247,88 @@ class StreamDecoder(KernelOps, nn.Module):
         ws = torch.empty(nws, dtype=torch.uint8, device=dev) if nws else None
         self._record("gated_delta", 4.0 * M * m.heads * m.dim * m.vdim, lambda: check(_lib.lib().evo_gated_delta_fwd(C.byref(gp), ptr(ws), nws, self._stream()), "evo_gated_delta_fwd"))
         return self._linear(out, pk["out"], M), pk["out"].Np
+
+    # ---- latent attention: m has heads, dim, rot_dim, vdim, kv_rank, rot_dims, scale, window (0: every earlier key)
+    def _pack_latent(self, m, uk, uv):
+        """Expansion of cache rows [latent | 0.. | rotated key part] into per-head keys [Uk_h c | rotated part] and values Uv_h c as one
+        linear layer: identity rows carry the shared rotated part into every head's key."""
+        dev, hd, rank_pad = uk.device, m.dim + m.rot_dim, _round_up(m.kv_rank, 8)
+        up = torch.zeros(m.heads * hd + m.heads * m.vdim, rank_pad + m.rot_dim, dtype=torch.bfloat16, device=dev)
+        for h in range(m.heads):
+            up[h * hd:h * hd + m.dim, :m.kv_rank] = uk[h * m.dim:(h + 1) * m.dim]
+            up[h * hd + m.dim:(h + 1) * hd, rank_pad:] = torch.eye(m.rot_dim, dtype=torch.bfloat16, device=dev)
+        up[m.heads * hd:, :m.kv_rank] = uv
+        expand = _Packed(up)
+        return {"expand": expand, "rank_pad": rank_pad, "cache_row": expand.Kp}
+
+    def _latent_prep(self, m, freq, rot_len, B, L, off, pos_dev, **part):
+        pp = LatentPrepParams(eps=self.config.eps, freq=freq.data_ptr() if freq is not None else None, rot_len=rot_len, B=B, L=L, H=m.heads, dim=m.dim, rot=m.rot_dim,
+                              rank=m.kv_rank, pos0=off, pos_dev=pos_dev.data_ptr() if pos_dev is not None else None, dtype=self._dt, rot_dims=m.rot_dims, **part)
+        hd, esz = m.dim + m.rot_dim, 4 if self._dt else 2
+        moved = (m.heads * (hd if part.get("dkv") else 2 * m.rot_dim) if part.get("q") else 0) + (2 * (m.kv_rank + m.rot_dim) if part.get("dkv") else 0) + 2 * part.get("q_rank", 0)
+        self._record("latent_prep", float(B * L) * moved * esz, lambda: check(_lib.lib().evo_latent_prep(C.byref(pp), self._stream()), "evo_latent_prep"))
+
+    def _latent_rows(self, r, m, lat, dkv_ptr, ld_dkv, norm_w, freq, rot_len, B, L, ip, off, pos_dev, q=None, query=None):
+        """Latents (normed) and turned key parts of the call's tokens -> rows of run r's cache, which is returned.  q (pointer, row
+        stride): queries whose rotated parts are turned in the same launch; query (pointer, row stride, norm weight, rank, out): the
+        queries' own latent, normed into out."""
+        row = lat["cache_row"]
+        cache = torch.zeros(B, L, row, dtype=self.act_dtype, device=self.device) if ip is None else self._kv_rows(ip, r, row, B, off, L, pos_dev)
+        part = dict(dkv=dkv_ptr, ld_dkv=ld_dkv, norm_w=norm_w.data_ptr(), cache=cache.data_ptr(), cache_row=row, cache_batch_stride=cache.shape[1] * row, rank_pad=lat["rank_pad"])
+        if q is not None:
+            part.update(q=q[0], ldq=q[1])
+        if query is not None:
+            part.update(dq=query[0], ld_dq=query[1], dq_norm_w=query[2].data_ptr(), q_rank=query[3], cq=query[4].data_ptr(), ld_cq=query[4].shape[1])
+        self._latent_prep(m, freq, rot_len, B, L, off, pos_dev, **part)
+        return cache
+
+    def _latent_turn(self, m, q, ldq, freq, rot_len, B, L, off, pos_dev):
+        """Turns the rotated parts of queries that were not there yet when the cache rows were written."""
+        if m.rot_dims:
+            self._latent_prep(m, freq, rot_len, B, L, off, pos_dev, q=q.data_ptr(), ldq=ldq)
+
+    @staticmethod
+    def _mean_keys(off, L, window):
+        """Keys that a query at positions off .. off + L - 1 sees on average."""
+        if window <= 0 or off + L <= window:
+            return off + (L + 1) / 2.0
+        ramp = max(0, min(L, window - off))           # queries whose window still reaches the sequence's start
+        return (ramp * (off + (ramp + 1) / 2.0) + (L - ramp) * float(window)) / L
+
+    def _latent_attend(self, m, lat, q_ptr, ldq, cache, uk, uv, gate_ptr, ld_gate, gate_per_channel, B, L, off, pos_dev):
+        """Prepared queries against the latent cache -> (B*L, heads*vdim padded), gated.  Steps and short portions stay in the latent space
+        (absorbed form); longer ones expand the visible rows into keys and values first."""
+        lib, dev, esz, M = _lib.lib(), cache.device, cache.element_size(), B * L
+        row, bstride, hd = lat["cache_row"], cache.shape[1] * lat["cache_row"], m.dim + m.rot_dim
+        pos_ptr = pos_dev.data_ptr() if pos_dev is not None else None
+        ldo = _round_up(m.heads * m.vdim, 64)
+        out = torch.empty(M, ldo, dtype=self.act_dtype, device=dev)
+        span = self._mean_keys(off, L, m.window)
+        if L <= ABSORBED_MAX_ROWS or pos_dev is not None:
+            dp = LatentDecodeParams(q=q_ptr, ldq=ldq, cache=cache.data_ptr(), cache_row=row, cache_batch_stride=bstride, rank_pad=lat["rank_pad"],
+                                    uk=uk.data_ptr(), uv=uv.data_ptr(), gate=gate_ptr, ld_gate=ld_gate, gate_per_channel=int(gate_per_channel),
+                                    out=out.data_ptr(), ldo=ldo, B=B, Lq=L, H=m.heads, dim=m.dim, rot=m.rot_dim, rank=m.kv_rank, vdim=m.vdim,
+                                    pos0=off, pos_dev=pos_ptr, window=m.window, scale=m.scale, dtype=self._dt,
+                                    max_keys=cache.shape[1] if pos_dev is not None else off + L)
+            nws = lib.evo_latent_attn_decode_workspace(C.byref(dp)) if self.latent_decode_path == "shared" else 0
+            ws = torch.empty(nws, dtype=torch.uint8, device=dev) if nws else None
+            # roofline bytes: each sequence's visible latents once (all heads share them)
+            self._record("latent_decode", float(M) * span * (m.kv_rank + m.rot_dim) * esz,
+                         lambda: check(lib.evo_latent_attn_decode(C.byref(dp), ptr(ws), nws, self._stream()), "evo_latent_attn_decode"))
+            return out
+        lo = max(0, off - (m.window - 1)) if m.window > 0 else 0
+        n, ex = off + L - lo, lat["expand"]
+        kv = torch.empty(B, n, ex.Np, dtype=self.act_dtype, device=dev)
+        for b in range(B):
+            self._linear(cache[b, lo:off + L], ex, n, out=kv[b])
+        ap = WindowAttnParams(q=q_ptr, q_tok_stride=ldq, gate=gate_ptr, gate_tok_stride=ld_gate, gate_per_head=0 if gate_per_channel else 1,
+                              k=kv.data_ptr() - lo * ex.Np * esz, v=kv.data_ptr() + (m.heads * hd - lo * ex.Np) * esz,
+                              k_tok_stride=ex.Np, v_tok_stride=ex.Np, k_batch_stride=n * ex.Np, v_batch_stride=n * ex.Np,
+                              out=out.data_ptr(), ldo=ldo, dtype=self._dt, B=B, Lq=L, H=m.heads, G=m.heads, dk=hd, dv=m.vdim, n_maps=1,
+                              q_pos0=off, window=m.window, keep_first=0, scale=m.scale, norm_eps=self.config.eps, out_scale=1.0)
+        self._record("window_attn", 2.0 * M * m.heads * span * (hd + m.vdim),
+                     lambda: check(lib.evo_window_attn_fwd(C.byref(ap), self._stream()), "evo_window_attn_fwd"))
+        return out
 
     def _run_chosen_experts(self, h, M, chosen, experts, ff, E, top, **act):
         """Only the chosen experts of a mixture: the (token, choice) pairs of `chosen` (M, top) int32 are sorted by expert, and every

@@ -450,6 +450,12 @@ typedef struct {
   int B; int64_t L; int H, dim, rot, rank;
   int64_t pos0; const int64_t* pos_dev; int dtype;
   int rot_dims;                               /* leading entries of a rotated part that are turned (even, <= rot) */
+  /* optional extensions (off when zero); q or dkv may be NULL then (that part is skipped):
+   *   rot_len: cosines and sines are multiplied by it (0: 1);
+   *   dq (B*L, q_rank): the queries' own latent; cq (B*L, ld_cq) = rms(dq) * dq_norm_w, columns [q_rank, ld_cq) zero. */
+  float rot_len;
+  const void* dq; int64_t ld_dq; const void* dq_norm_w; int q_rank;
+  void* cq; int64_t ld_cq;
 } evo_latent_prep_params;
 int evo_latent_prep(const evo_latent_prep_params* p, void* stream);
 
@@ -466,6 +472,7 @@ typedef struct {
   int B; int64_t Lq; int H, dim, rot, rank, vdim;
   int64_t pos0; const int64_t* pos_dev; int64_t window; float scale; int dtype;
   int64_t max_keys;                           /* host bound on the keys a query can see (sizes the key splits); 0: unknown */
+  int gate_per_channel;                       /* 1: gate is (B*Lq, H*vdim), one number per output channel */
 } evo_latent_decode_params;
 /* workspace: evo_latent_attn_decode_workspace() bytes (absorbed queries and per-split partial sums); with less, the per-head kernel runs */
 size_t evo_latent_attn_decode_workspace(const evo_latent_decode_params* p);
@@ -686,6 +693,32 @@ typedef struct {
 size_t evo_gla_workspace(const evo_gla_params* p);
 int evo_gla_fwd(const evo_gla_params* p, void* workspace, size_t workspace_bytes, void* stream);
 
+/* ==== designs that mix latent attention, windowed attention with shared keys and values, and linear attention with a constant decay
+ * per head (Nilatar).  Same conventions: `dtype` 0 = bf16 activations, 1 = fp32; weights and parameter vectors bf16. ==== */
+
+/* out (n, D) fp32 = table[id] * scale */
+int evo_embed_scaled_f32(const void* ids, int ids_are_i64, const void* table, float* out, int64_t n_tokens, int D, int vocab, float scale, void* stream);
+
+/* Linear attention with one constant decay per head, per head h over q, k (H*dk) and v (H*dv) of a row (act 1: each through silu first):
+ *   S <- decay[h] S + k v^T;   y = S^T (q q_scale)        decay (H) fp32, y (rows, H*dv) fp32
+ * state (B, H, dk, dv) fp32 (zero_start: starts at 0; NULL: starts at 0 and is not kept).
+ * recurrent: 1 = token by token whatever the shape (comparisons); otherwise prompts in bf16 run block-wise on the tensor cores.
+ * workspace: evo_decay_scan_workspace() bytes. */
+typedef struct {
+  const void* q; const void* k; const void* v; int64_t ld;
+  const float* decay; int act; float q_scale;
+  float* state; int zero_start;
+  float* y;
+  int dtype;
+  int B; int64_t L; int H, dk, dv;
+  int recurrent;
+} evo_decay_scan_params;
+size_t evo_decay_scan_workspace(const evo_decay_scan_params* p);
+int evo_decay_scan_fwd(const evo_decay_scan_params* p, void* workspace, size_t workspace_bytes, void* stream);
+
+/* out = rms(y) * norm_w * sigmoid(gate): the row's `width` values are normed together; y (rows, width) fp32, gate (rows, ldg) and
+ * out (rows, ldo) activations, columns [width, ldo) zero. */
+int evo_norm_gate(const float* y, const void* gate, int64_t ldg, const void* norm_w, void* out, int64_t ldo, int64_t rows, int width, float eps, int dtype, void* stream);
 
 #ifdef __cplusplus
 }
