@@ -1,6 +1,6 @@
 """bench.py — nucleotides/sec of the Evo-1 7B forward on B200 (BASELINE.json metric).
 
-    python bench.py [--gpus N] [--steps K] [--warmup W] [--workload 8k|131k|1k|32k|gen|zaverax|movalorn|nelovik|gakupel|gagotar] [--impl ours|reference]
+    python bench.py [--gpus N] [--steps K] [--warmup W] [--workload 8k|131k|1k|32k|gen|zaverax|movalorn|nelovik|gakupel|gagotar|nilatar] [--impl ours|reference]
 
 Workload "8k" (default): evo-1-8k-base scoring forward, batch 8 x
 8192 nt of synthetic uniform ACGT (+BOS => L = 8193), bf16, random-init weights of the 7B
@@ -13,7 +13,8 @@ collective (weak scaling); "131k" runs the sequence-parallel forward instead.
 Workload "zaverax" (an option; the default workload and its JSON contract are unchanged): the Zaverax design beside StripedHyena at
 equal layer sizes, prefill and decode, with a per-kernel roofline breakdown (bench_arch).  Workload "movalorn": the same for the
 Movalorn design beside Zaverax, the closest family.  Workload "nelovik": the Nelovik design beside Zaverax likewise.  Workload "gakupel":
-the Gakupel design beside Nelovik.  Workload "gagotar": the Gagotar design beside Gakupel.
+the Gakupel design beside Nelovik.  Workload "gagotar": the Gagotar design beside Gakupel.  Workload "nilatar": the Nilatar design
+beside Gagotar and Movalorn, the two families that share its parts.
 --impl reference: the reference's own CPU implementation of the path.  stripedhyena==0.2.2 is
 not installable offline, so this arm times the oracle restatement (kind "port") on the host
 cores, rank 0 only, on a bounded sample of the same workload.
@@ -703,6 +704,31 @@ def _gagotar_models(size, dev):
     return Gagotar(GagotarConfig.from_dict(gc)).init_random(0, device=dev), gk
 
 
+def _nilatar_models(size, dev):
+    """A Nilatar model between the two families that share its parts -- Gagotar (pre-norm with layer scales, linear attention with a matrix
+    state) and Movalorn (latent attention, dense feed-forwards) -- of equal width, depth and head count, random weights.  Nilatar: latent
+    attention (heads of 64 + 64 query and 128 value channels, latents of 512 for the keys and 768 for the queries, over the whole prompt),
+    linear attention with heads of 128 x 128, windowed sink attention (heads of 128 / 128, a fourth as many key heads, 1024 positions) and
+    a second such layer that reads the first one's keys and values; dense feed-forwards of Movalorn's width, none behind the linear attention."""
+    from evo_b200.nilatar import Nilatar, NilatarConfig
+    s = ARCH_SIZES[size]
+    d, H = s["width"], s["heads"]
+    ff = (8 * d // 3 + 255) // 256 * 256
+    gt, gk = _gagotar_models(size, dev)
+    del gk
+    mv, zv = _movalorn_models(size, dev)
+    del zv
+    dense = {"kind": "dense", "ff": ff}
+    win = {"heads": H, "kv_heads": H // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024}}
+    lat = {"heads": H, "dim": 64, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": 768, "scale": 128 ** -0.5,
+           "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    lin = {"heads": H, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-2.0 - 6.0 * h / H) for h in range(H)]}
+    nc = {"architecture": "Nilatar", "vocab": 512, "width": d, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0},
+          "layers": [{"type": "attention", "mixer": win, "mlp": dense}, {"type": "latent_attention", "mixer": lat, "mlp": dense},
+                     {"type": "lightning", "mixer": lin, "mlp": None}, {"type": "attention", "mixer": dict(win, kv_from=0), "mlp": dense}]}
+    return Nilatar(NilatarConfig.from_dict(nc)).init_random(0, device=dev), [("gagotar", gt), ("movalorn", mv)]
+
+
 def bench_arch(args):
     """--workload zaverax: prefill and decode throughput of the Zaverax design beside StripedHyena at equal layer sizes (random
     weights, 4 layers each, one of them attention), with a per-kernel breakdown against the measured rooflines.  Inputs are larger
@@ -718,16 +744,17 @@ def bench_arch(args):
              "window_attn": ("flop/s", peaks["bf16_tflops"] * 1e12), "hgrn2": ("fp32 lane-op/s", fp32_lane_ops),
              "gated_delta": ("fp32 lane-op/s", fp32_lane_ops), "ssd": ("fp32 lane-op/s", fp32_lane_ops), "mlstm": ("fp32 lane-op/s", fp32_lane_ops), "gla": ("fp32 lane-op/s", fp32_lane_ops), "mixed_attn": ("flop/s", peaks["bf16_tflops"] * 1e12)}
     family = args.workload
-    other = {"zaverax": "stripedhyena", "movalorn": "zaverax", "nelovik": "zaverax", "gakupel": "nelovik", "gagotar": "gakupel"}[family]
-    bound.update({"mingru": ("B/s", peaks["hbm_gbs"] * 1e9), "latent_decode": ("B/s", peaks["hbm_gbs"] * 1e9)})
+    other = {"zaverax": "stripedhyena", "movalorn": "zaverax", "nelovik": "zaverax", "gakupel": "nelovik", "gagotar": "gakupel", "nilatar": "gagotar and movalorn"}[family]
+    bound.update({"decay_scan": ("B/s", peaks["hbm_gbs"] * 1e9), "mingru": ("B/s", peaks["hbm_gbs"] * 1e9), "latent_decode": ("B/s", peaks["hbm_gbs"] * 1e9)})
     out = {"workload": family, "metric": f"tokens/sec, prefill and decode, {family} beside {other} at equal sizes", "unit": "tok/s", "dtype": "bf16",
            "data": "synthetic", "steps": steps, "warmup": warmup, "peaks": peaks, "sizes": {}}
     launches = 0
     with ClockSampler(0) as clocks:
         for size, s in ARCH_SIZES.items():
-            zv, sh = {"zaverax": _arch_models, "movalorn": _movalorn_models, "nelovik": _nelovik_models, "gakupel": _gakupel_models, "gagotar": _gagotar_models}[family](size, dev)
+            zv, sh = {"zaverax": _arch_models, "movalorn": _movalorn_models, "nelovik": _nelovik_models, "gakupel": _gakupel_models, "gagotar": _gagotar_models, "nilatar": _nilatar_models}[family](size, dev)
+            others = sh if isinstance(sh, list) else [(other, sh)]
             rec = {}
-            for name, model in ((family, zv), (other, sh)):
+            for name, model in [(family, zv)] + others:
                 B, L = s["prefill"]
                 ids = torch.randint(0, 512, (B, L), device=dev)
                 fwd = lambda: model(ids)
@@ -784,7 +811,7 @@ def bench_arch(args):
                 del d, lg
                 torch.cuda.empty_cache()
             out["sizes"][size] = rec
-            del zv, sh
+            del zv, sh, others, model
             torch.cuda.empty_cache()
     out["value"] = out["sizes"]["4k"][family]["prefill_tok_s"]
     out["n_gpus"] = 1
@@ -800,14 +827,14 @@ def main():
     ap.add_argument("--steps", type=int, default=None)
     ap.add_argument("--warmup", type=int, default=None)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="8k", choices=list(WORKLOADS) + ["zaverax", "movalorn", "nelovik", "gakupel", "gagotar"])
+    ap.add_argument("--workload", default="8k", choices=list(WORKLOADS) + ["zaverax", "movalorn", "nelovik", "gakupel", "gagotar", "nilatar"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-sub", action="store_true", help="default workload only: skip the sp131k / gen sub-records")
     ap.add_argument("--no-gen", action="store_true", help="skip the cached-generation sub-record")
     ap.add_argument("--sub-steps", type=int, default=3, help="timed steps of the 131k sub-record")
     ap.add_argument("--gen-tokens", type=int, default=None, help="new tokens of the end-to-end generate() run (default: 4096 = BASELINE configs[3])")
     args = ap.parse_args()
-    if args.workload in ("zaverax", "movalorn", "nelovik", "gakupel", "gagotar"):
+    if args.workload in ("zaverax", "movalorn", "nelovik", "gakupel", "gagotar", "nilatar"):
         return bench_arch(args)
     wl = WORKLOADS[args.workload]
     if args.impl == "reference":

@@ -13,6 +13,7 @@ LIB_PATH = os.path.join(_HERE, "libevo_b200.so")
 EPI_NONE, EPI_BIAS, EPI_BIAS_RESID, EPI_RESID, EPI_GELU_GATE = range(5)
 EPI_BIAS_ROPE = 6
 EPI_HYENA_STEP = 7
+EPI_SILU_COLS, EPI_GELU_TANH_GATE = 8, 9
 
 
 class EvoError(RuntimeError):
@@ -24,7 +25,7 @@ class GemmParams(C.Structure):
                 ("bias", C.c_void_p), ("residual", C.c_void_p), ("ldr", C.c_int64),
                 ("M", C.c_int64), ("N", C.c_int64), ("K", C.c_int64), ("epilogue", C.c_int), ("variant", C.c_int),
                 ("rope_cos", C.c_void_p), ("rope_sin", C.c_void_p), ("rope_L", C.c_int64), ("rope_cols", C.c_int64),
-                ("c_peers", C.c_void_p), ("n_c_peers", C.c_int), ("peer_period", C.c_int64), ("peer_inner", C.c_int64), ("peer_row0", C.c_int64)]
+                ("c_peers", C.c_void_p), ("n_c_peers", C.c_int), ("peer_period", C.c_int64), ("peer_inner", C.c_int64), ("peer_row0", C.c_int64), ("act_cols", C.c_int64)]
 
 
 class GemmSmallMParams(C.Structure):
@@ -33,7 +34,7 @@ class GemmSmallMParams(C.Structure):
                 ("M", C.c_int64), ("N", C.c_int64), ("K", C.c_int64), ("epilogue", C.c_int),
                 ("workspace", C.c_void_p), ("workspace_bytes", C.c_size_t),
                 ("fir_state", C.c_void_p), ("state", C.c_void_p), ("fir_w", C.c_void_p), ("fir_b", C.c_void_p), ("Dskip", C.c_void_p),
-                ("poles", C.c_void_p), ("residues", C.c_void_p)]
+                ("poles", C.c_void_p), ("residues", C.c_void_p), ("act_cols", C.c_int64)]
 
 
 class HyenaParams(C.Structure):
@@ -204,7 +205,7 @@ class MlstmParams(C.Structure):
 class GluActParams(C.Structure):
     _fields_ = [("gate", C.c_void_p), ("up", C.c_void_p), ("ld", C.c_int64), ("out", C.c_void_p), ("ldo", C.c_int64), ("rows", C.c_int64), ("F", C.c_int), ("act", C.c_int),
                 ("group_w", C.c_void_p), ("ldw", C.c_int64), ("group", C.c_int), ("n_groups", C.c_int), ("tail_w", C.c_int),
-                ("dtype", C.c_int), ("limit", C.c_float), ("slope", C.c_float)]
+                ("dtype", C.c_int), ("limit", C.c_float), ("slope", C.c_float), ("interleave", C.c_int)]
 
 
 class MixedAttnParams(C.Structure):
@@ -227,7 +228,7 @@ class GlaParams(C.Structure):
 class DecayScanParams(C.Structure):
     _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("ld", C.c_int64), ("decay", C.c_void_p), ("act", C.c_int), ("q_scale", C.c_float),
                 ("state", C.c_void_p), ("zero_start", C.c_int), ("y", C.c_void_p), ("dtype", C.c_int),
-                ("B", C.c_int), ("L", C.c_int64), ("H", C.c_int), ("dk", C.c_int), ("dv", C.c_int), ("recurrent", C.c_int)]
+                ("B", C.c_int), ("L", C.c_int64), ("H", C.c_int), ("dk", C.c_int), ("dv", C.c_int), ("recurrent", C.c_int), ("part_len", C.c_int64)]
 
 
 # name -> (restype, argtypes); every symbol include/evo_b200.h declares

@@ -48,6 +48,7 @@ struct SmArgs {
   const bf16* fir_w; const bf16* fir_b; const bf16* Dskip;
   const float* poles; const float* residues;
   int D;
+  long long act_cols;               // EVO_EPI_SILU_COLS
   int* counters;                    // [n_tiles], zero between launches
   float* slots;                     // [2 * gridDim.x][R * Mb][128] fp32 partials
   long long* trace;                 // debug: [gridDim.x][16] time stamps (evo_debug_smallm_trace), NULL normally
@@ -58,6 +59,8 @@ long long* g_trace = nullptr;
 __device__ __forceinline__ long long gtimer() { long long t; asm volatile("mov.u64 %0, %%globaltimer;" : "=l"(t)); return t; }
 __device__ __forceinline__ void stamp(const SmArgs& g, int i) { if (g.trace) g.trace[blockIdx.x * 16 + i] = clock64(); }
 
+__device__ __forceinline__ float gelu_tanh(float z) { return __fdividef(z, 1.f + __expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z))); }
+__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 __device__ __forceinline__ float gelu_erf(float x) { return 0.5f * x * (1.0f + erff(x * 0.70710678118654752440f)); }
 __device__ __forceinline__ void named_bar(int id, int n) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(n) : "memory"); }
 
@@ -102,6 +105,10 @@ __device__ __forceinline__ void finalize16(const SmArgs& g, long long n, int b0,
     float o;
     if constexpr (EPI == EVO_EPI_GELU_GATE) {
       o = rbf(gelu_erf(rbf(v0[j]))) * rbf(v1[j]);
+    } else if constexpr (EPI == EVO_EPI_GELU_TANH_GATE) {
+      o = gelu_tanh(v0[j]) * v1[j];
+    } else if constexpr (EPI == EVO_EPI_SILU_COLS) {
+      o = n < g.act_cols ? silu(v0[j]) : v0[j];
     } else {
       o = v0[j];
       if constexpr (EPI == EVO_EPI_BIAS || EPI == EVO_EPI_BIAS_RESID) o += bias;
@@ -112,7 +119,7 @@ __device__ __forceinline__ void finalize16(const SmArgs& g, long long n, int b0,
 }
 
 constexpr int EPI_HYENA_STEP = 7;   // EVO_EPI_HYENA_STEP
-template <int EPI> struct RowGroups { static constexpr int R = EPI == EVO_EPI_GELU_GATE ? 2 : (EPI == EPI_HYENA_STEP ? 3 : 1); };
+template <int EPI> struct RowGroups { static constexpr int R = EPI == EVO_EPI_GELU_GATE || EPI == EVO_EPI_GELU_TANH_GATE ? 2 : (EPI == EPI_HYENA_STEP ? 3 : 1); };
 
 // One decode step of the Hyena operator for channel `ch` of head `tile`, 16 batch rows: the arithmetic of hyena_step_kernel
 // (hyena.cu; engine.step_fir + step_iir of the reference) on the in-projection's fp32 sums z2/z1/zv (x2, x1, v rows of the head).
@@ -416,6 +423,7 @@ int launch(const evo_gemm_smallm_params* p, cudaStream_t st) {
   g.M = (int)p->M; g.Mb = Mb;
   g.fir_state = (bf16*)p->fir_state; g.state = p->state; g.fir_w = (const bf16*)p->fir_w; g.fir_b = (const bf16*)p->fir_b; g.Dskip = (const bf16*)p->Dskip;
   g.poles = p->poles; g.residues = p->residues; g.D = (int)(p->N / 3);
+  g.act_cols = p->act_cols;
   g.n_tiles = (int)(p->N / (R * WROWS));
   g.KB = (int)(p->K / BK);
   const int stage_bytes = R * WROWS * BK * 2 + Mb * BK * 2;
@@ -459,7 +467,7 @@ extern "C" void evo_debug_smallm_trace(void* buf) { g_trace = (long long*)buf; }
 
 extern "C" size_t evo_gemm_smallm_workspace(int64_t M, int64_t N, int64_t K, int epilogue) {
   (void)K;
-  const int R = epilogue == EVO_EPI_GELU_GATE ? 2 : (epilogue == EPI_HYENA_STEP ? 3 : 1);
+  const int R = epilogue == EVO_EPI_GELU_GATE || epilogue == EVO_EPI_GELU_TANH_GATE ? 2 : (epilogue == EPI_HYENA_STEP ? 3 : 1);
   const size_t Mb = (size_t)((M + 15) / 16 * 16);
   if (N / (R * WROWS) > 4096) return 0;
   return 16384 + (size_t)2 * device_sm_count() * R * Mb * WROWS * sizeof(float);
@@ -481,6 +489,8 @@ extern "C" int evo_gemm_smallm(const evo_gemm_smallm_params* p, void* stream) {
     case EVO_EPI_BIAS_RESID: return launch<EVO_EPI_BIAS_RESID>(p, (cudaStream_t)stream);
     case EVO_EPI_RESID: return launch<EVO_EPI_RESID>(p, (cudaStream_t)stream);
     case EVO_EPI_GELU_GATE: return launch<EVO_EPI_GELU_GATE>(p, (cudaStream_t)stream);
+    case EVO_EPI_GELU_TANH_GATE: return launch<EVO_EPI_GELU_TANH_GATE>(p, (cudaStream_t)stream);
+    case EVO_EPI_SILU_COLS: return launch<EVO_EPI_SILU_COLS>(p, (cudaStream_t)stream);
     case EPI_HYENA_STEP:
       EVO_REQUIRE(p->bias && p->fir_state && p->state && p->fir_w && p->fir_b && p->Dskip && p->poles && p->residues, "evo_gemm_smallm: EVO_EPI_HYENA_STEP needs bias, states and filter parameters");
       EVO_REQUIRE(p->N % (3 * WROWS) == 0, "evo_gemm_smallm: EVO_EPI_HYENA_STEP needs N = 3 * heads * 128");

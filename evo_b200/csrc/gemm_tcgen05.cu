@@ -61,6 +61,7 @@ struct GemmArgs {
   // c_peer[(n % peer_period) / peer_inner] at [(peer_row0 + m) * ldc + (n / peer_period) * peer_inner + n % peer_inner]
   bf16* c_peer[8]; int n_peers; int peer_period, peer_inner; long long peer_row0;
   const bf16* rope_cos; const bf16* rope_sin;   // EVO_EPI_BIAS_ROPE: (positions, 64) bf16 tables, row l = position of token row l
+  long long act_cols;                           // EVO_EPI_SILU_COLS
   long long rope_L, rope_cols;                  //   rows repeat with period rope_L (tokens per sequence); columns < rope_cols (q and k) are rotated
   const long long* targets;   // EPI_LSE only: (M) target token per row (-1: none)
   float4* part;               // EPI_LSE only: (M, n_blocks) per-row partial statistics {max, sum e^(x-max), sum e^(x-max) x, target logit}
@@ -75,6 +76,9 @@ struct GemmArgs {
 
 constexpr int EPI_LSE = 5;     // internal: scoring epilogue (evo_unembed_score); no C is written (EVO_EPI_BIAS_ROPE is 6)
 
+// tanh-form gelu as z * sigmoid(2 sqrt(2/pi) (z + 0.044715 z^3)), and silu
+__device__ __forceinline__ float gelu_tanh(float z) { return __fdividef(z, 1.f + __expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z))); }
+__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 __device__ __forceinline__ float gelu_erf(float x) { return 0.5f * x * (1.0f + erff(x * 0.70710678118654752440f)); }
 
 // grouped rasterisation: GROUP_M row-blocks share the sweep over n so their A tiles stay in L2
@@ -111,6 +115,10 @@ __device__ __forceinline__ void store_chunk(const GemmArgs& g, long long row, in
       float b0 = rbf(__uint_as_float(acc2[2 * j])), b1 = rbf(__uint_as_float(acc2[2 * j + 1]));
       outw[j] = pack_bf16(rbf(gelu_erf(a0)) * b0, rbf(gelu_erf(a1)) * b1);
     }
+  } else if constexpr (EPI == EVO_EPI_GELU_TANH_GATE) {
+#pragma unroll
+    for (int j = 0; j < 16; ++j)
+      outw[j] = pack_bf16(gelu_tanh(__uint_as_float(acc[2 * j])) * __uint_as_float(acc2[2 * j]), gelu_tanh(__uint_as_float(acc[2 * j + 1])) * __uint_as_float(acc2[2 * j + 1]));
   } else {
     float v[32];
 #pragma unroll
@@ -137,6 +145,11 @@ __device__ __forceinline__ void store_chunk(const GemmArgs& g, long long row, in
           v[q * 8 + 2 * j + 1] = rbf(v[q * 8 + 2 * j + 1]) + bf_hi(rw[j]);
         }
       }
+    }
+    if constexpr (EPI == EVO_EPI_SILU_COLS) {
+      const long long act = g.act_cols - col;              // how many of the 32 columns go through the activation
+#pragma unroll
+      for (int j = 0; j < 32; ++j) if (j < act) v[j] = silu(v[j]);
     }
 #pragma unroll
     for (int j = 0; j < 16; ++j) outw[j] = pack_bf16(v[2 * j], v[2 * j + 1]);
@@ -196,7 +209,8 @@ template <int CG, int EPI, int BN>
 __global__ void __launch_bounds__(NTHREADS, (BN == BN_SMALL ? 2 : 1))
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const GemmArgs g) {
   using C_ = Cfg<CG, BN>;
-  static_assert(EPI != EVO_EPI_GELU_GATE || BN == BN_BIG, "the gate epilogue needs [l1 | l2] halves of a 256-column tile");
+  constexpr bool GATE = EPI == EVO_EPI_GELU_GATE || EPI == EVO_EPI_GELU_TANH_GATE;
+  static_assert(!GATE || BN == BN_BIG, "the gate epilogue needs [l1 | l2] halves of a 256-column tile");
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   constexpr bool SMALL = BN == BN_SMALL;
@@ -392,7 +406,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
             if (row < g.M) store_rope_pair(g, row, n_blk * BN + hc + c, l, c, rotate, r1, r2);
           }
         }
-      } else if constexpr (EPI == EVO_EPI_GELU_GATE && BN == BN_BIG) {
+      } else if constexpr (GATE && BN == BN_BIG) {
 #pragma unroll 1
         for (int c = 0; c < BN / 2; c += 32) {
           uint32_t r1[32], r2[32];
@@ -444,7 +458,7 @@ int launch(const evo_gemm_params* p, cudaStream_t st, const long long* targets =
   g.targets = targets; g.part = part;
   g.n_peers = p->n_c_peers; g.peer_period = (int)p->peer_period; g.peer_inner = (int)p->peer_inner; g.peer_row0 = p->peer_row0;
   for (int i = 0; i < 8; ++i) g.c_peer[i] = i < p->n_c_peers ? (bf16*)p->c_peers[i] : nullptr;
-  g.rope_cos = (const bf16*)p->rope_cos; g.rope_sin = (const bf16*)p->rope_sin; g.rope_L = p->rope_L > 0 ? p->rope_L : 1; g.rope_cols = p->rope_cols;
+  g.rope_cos = (const bf16*)p->rope_cos; g.rope_sin = (const bf16*)p->rope_sin; g.rope_L = p->rope_L > 0 ? p->rope_L : 1; g.rope_cols = p->rope_cols; g.act_cols = p->act_cols;
   g.a_rows = a_rows;
   g.b_tiled = b_tiled;
   // small tile: two 64-column k-blocks per barrier round when K allows (halves the issue thread's serial rounds)
@@ -542,6 +556,10 @@ int dispatch_epi(const evo_gemm_params* p, cudaStream_t st) {
     case EVO_EPI_BIAS_ROPE:
       if constexpr (BN == BN_BIG) return launch<CG, EVO_EPI_BIAS_ROPE, BN>(p, st);
       else { set_error("evo_gemm: the rotary epilogue is not available on the small-M tile (variant 2)"); return -1; }
+    case EVO_EPI_SILU_COLS: return launch<CG, EVO_EPI_SILU_COLS, BN>(p, st);
+    case EVO_EPI_GELU_TANH_GATE:
+      if constexpr (BN == BN_BIG) return launch<CG, EVO_EPI_GELU_TANH_GATE, BN>(p, st);
+      else { set_error("evo_gemm: the GELU-gate epilogue is not available on the small-M tile (variant 2)"); return -1; }
     case EVO_EPI_GELU_GATE:
       if constexpr (BN == BN_BIG) return launch<CG, EVO_EPI_GELU_GATE, BN>(p, st);
       else { set_error("evo_gemm: the GELU-gate epilogue is not available on the small-M tile (variant 2)"); return -1; }

@@ -570,7 +570,7 @@ __device__ __forceinline__ float glu_value(float z, float u, int act, float limi
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) glu_act_kernel(const T* __restrict__ g, const T* __restrict__ u, int64_t ld, T* __restrict__ out, int64_t ldo,
                                                       int F, int act, const float* __restrict__ group_w, int64_t ldw, int group, int n_groups, int tail_w,
-                                                      float limit, float slope) {
+                                                      float limit, float slope, int il) {
   const int64_t r = blockIdx.x;
   const T* gr = g + r * ld; const T* ur = u ? u + r * ld : nullptr;
   T* orow = out + r * ldo;
@@ -586,11 +586,13 @@ __global__ void __launch_bounds__(256) glu_act_kernel(const T* __restrict__ g, c
     if (wr) { const int e = c / group; if (e < n_groups) wt = wr[e]; else if (tail_w) wt = wr[n_groups]; }
     if (wt != 0.f) {
       if (VEC) {
-        const float4 g4 = ld4(gr + c), u4 = ur ? ld4(ur + c) : make_float4(1.f, 1.f, 1.f, 1.f);
+        const int64_t cc = il > 0 ? (int64_t)(c / il) * 2 * il + c % il : c;
+        const float4 g4 = ld4(gr + cc), u4 = ur ? ld4(ur + cc) : make_float4(1.f, 1.f, 1.f, 1.f);
         v[0] = glu_value<T>(g4.x, u4.x, act, limit, slope) * wt; v[1] = glu_value<T>(g4.y, u4.y, act, limit, slope) * wt;
         v[2] = glu_value<T>(g4.z, u4.z, act, limit, slope) * wt; v[3] = glu_value<T>(g4.w, u4.w, act, limit, slope) * wt;
       } else {
-        v[0] = glu_value<T>(ldf(gr + c), ur ? ldf(ur + c) : 1.f, act, limit, slope) * wt;
+        const int64_t cc = il > 0 ? (int64_t)(c / il) * 2 * il + c % il : c;
+        v[0] = glu_value<T>(ldf(gr + cc), ur ? ldf(ur + cc) : 1.f, act, limit, slope) * wt;
       }
     }
   }
@@ -636,6 +638,7 @@ extern "C" int evo_branch_norm(const evo_branch_norm_params* p, void* stream) {
 
 extern "C" int evo_glu_act_ex(const evo_glu_act_params* p, void* stream) {
   EVO_REQUIRE(p->gate && p->out && p->F > 0 && p->ldo >= p->F && p->act >= 0 && p->act <= 3, "evo_glu_act: bad arguments");
+  EVO_REQUIRE(p->interleave >= 0 && p->interleave % 4 == 0, "evo_glu_act: interleave must be a multiple of 4");
   EVO_REQUIRE(p->act != 3 || (p->up && p->limit > 0.f), "evo_glu_act: the limited form needs both factors and a positive limit");
   EVO_REQUIRE(p->group_w == nullptr || (p->group > 0 && p->n_groups > 0 && p->ldw >= p->n_groups + (p->tail_w ? 1 : 0)), "evo_glu_act: bad groups");
   if (p->rows == 0) return 0;
@@ -648,7 +651,7 @@ extern "C" int evo_glu_act_ex(const evo_glu_act_params* p, void* stream) {
   cudaStream_t st = (cudaStream_t)stream;
 #define EVO_GLU(TT, V) \
   glu_act_kernel<TT, V><<<grid, block, 0, st>>>((const TT*)p->gate, (const TT*)p->up, p->ld, (TT*)p->out, p->ldo, p->F, p->act, p->group_w, p->ldw, p->group, p->n_groups, \
-                                                p->tail_w, p->limit, p->slope)
+                                                p->tail_w, p->limit, p->slope, p->interleave)
   if (p->dtype) { if (vec) EVO_GLU(float, true); else EVO_GLU(float, false); }
   else { if (vec) EVO_GLU(bf16, true); else EVO_GLU(bf16, false); }
 #undef EVO_GLU

@@ -11,7 +11,8 @@ trace replay and command line drive it.  State, keyed by RUN index r:
                                         layer's keys and values has no entry
     d["hyena"].state_dict[r]            (B, heads, dim, vdim) fp32: the linear attention's matrix state
 Cache rows stay where they are; the window only limits what the kernels read.  Closing one sublayer and opening the next is ONE row kernel
-(evo_sum_norm), and all projections that read the mixer's input are one GEMM.  Linear layers: bf16 activations -> the framework's tcgen05
+(evo_sum_norm), all projections that read the mixer's input are one GEMM, and the feed-forward's gate and the linear attention's silu sit
+in their GEMMs' epilogues.  Linear layers: bf16 activations -> the framework's tcgen05
 GEMMs (weights zero-padded once to their tiles); fp32 activations (dtype=torch.float32) -> evo_gemm_simt, true fp32 multiply-add.
 """
 from __future__ import annotations
@@ -23,10 +24,8 @@ import torch
 
 from .. import _lib
 from .._lib import DecayScanParams, WindowAttnParams, check, ptr
-from ..stream_model import StreamDecoder, _Packed, _round_up
+from ..stream_model import StreamDecoder, _Packed, _PackedGate, _round_up
 from .config import NilatarConfig
-
-ACT_GELU_TANH = 0
 
 
 class Nilatar(StreamDecoder):
@@ -87,7 +86,7 @@ class Nilatar(StreamDecoder):
                 e["decay"] = torch.tensor(m.decay, dtype=torch.float64).to(torch.float32).to(dev)
             if layer.ff:
                 q = f"l{i}.mlp."
-                e["up"], e["down"] = _Packed(torch.cat([w[q + "gate"], w[q + "up"]], 0)), _Packed(w[q + "down"])
+                e["up"], e["down"] = _PackedGate(w[q + "gate"], w[q + "up"]), _Packed(w[q + "down"], _PackedGate.RUN)
             packed["layers"].append(e)
         self._packed = packed
         return packed
@@ -135,32 +134,30 @@ class Nilatar(StreamDecoder):
         return self._linear(out, pk["out"], M), pk["out"].Np
 
     def _lightning(self, r, i, m, h, B, L, rec, fresh):
-        """silu of the projections and the recurrence (evo_decay_scan_fwd), norm over all heads and gate -> output projection."""
+        """silu of the projections (in the GEMM's epilogue, or in the recurrence), the recurrence, norm over all heads and gate -> output projection."""
         pk, w, lib = self._packed["layers"][i], self.weights, _lib.lib()
         M, dev = B * L, h.device
-        z = self._linear(h, pk["in"], M)
-        esz, ldz, col = z.element_size(), pk["in"].Np, pk["col"]
+        col, ldz, vw = pk["col"], pk["in"].Np, m.heads * m.vdim
+        z = self._linear(h, pk["in"], M, silu_cols=col["g"] if self._fused else 0)
+        esz = z.element_size()
         at = lambda n: z.data_ptr() + col[n] * esz
-        vw = m.heads * m.vdim
         state, zero = self._matrix_state(r, rec, B, m.heads, m.dim, m.vdim, fresh)
         y = torch.empty(M, vw, dtype=torch.float32, device=dev)
-        sp = DecayScanParams(q=at("q"), k=at("k"), v=at("v"), ld=ldz, decay=pk["decay"].data_ptr(), act=1, q_scale=1.0, state=state.data_ptr(), zero_start=zero,
+        sp = DecayScanParams(q=at("q"), k=at("k"), v=at("v"), ld=ldz, decay=pk["decay"].data_ptr(), act=int(not self._fused), q_scale=1.0, state=state.data_ptr(), zero_start=zero,
                              y=y.data_ptr(), dtype=self._dt, B=B, L=L, H=m.heads, dk=m.dim, dv=m.vdim, recurrent=self.decay_recurrent)
         nws = lib.evo_decay_scan_workspace(C.byref(sp))
         ws = torch.empty(nws, dtype=torch.uint8, device=dev) if nws else None
-        self._record("decay_scan", 3.0 * M * m.heads * m.dim * m.vdim, lambda: check(lib.evo_decay_scan_fwd(C.byref(sp), ptr(ws), nws, self._stream()), "evo_decay_scan_fwd"))
+        # roofline bytes: the projections once, the fp32 read-outs once
+        self._record("decay_scan", float(M) * m.heads * ((2 * m.dim + m.vdim) * esz + 4 * m.vdim), lambda: check(lib.evo_decay_scan_fwd(C.byref(sp), ptr(ws), nws, self._stream()), "evo_decay_scan_fwd"))
         ldo = _round_up(vw, 64)
         out = torch.empty(M, ldo, dtype=self.act_dtype, device=dev)
         self._record("norm_gate", float(M) * vw * (4.0 + 2.0 * esz), lambda: check(lib.evo_norm_gate(
             ptr(y), C.c_void_p(at("g")), ldz, ptr(w[f"l{i}.mix.norm"]), ptr(out), ldo, M, vw, self.config.eps, self._dt, self._stream()), "evo_norm_gate"))
         return self._linear(out, pk["out"], M), pk["out"].Np
 
-    def _feed_forward(self, i, ff, h, M):
+    def _feed_forward(self, i, h, M):
         pk = self._packed["layers"][i]
-        z = self._linear(h, pk["up"], M)
-        a = torch.empty(M, pk["down"].Kp, dtype=self.act_dtype, device=h.device)
-        self._glu(z.data_ptr(), z.data_ptr() + ff * z.element_size(), pk["up"].Np, a, pk["down"].Kp, M, ff, ACT_GELU_TANH)
-        return self._linear(a, pk["down"], M), pk["down"].Np
+        return self._linear(self._gelu_gate(h, pk["up"], M), pk["down"], M), pk["down"].Np
 
     def _body(self, ids, B, L, ipd, off: int, pos_dev=None, rows=None):
         """embed -> every layer -> final norm -> head.  Returns fp32 logits (B*L, V), or (len(rows), V) for the flat row
@@ -194,7 +191,7 @@ class Nilatar(StreamDecoder):
             branches, scale = [(y, ldy, None, 1.0)], w[f"l{i}.ls1"]
             if layer.ff:
                 h = open_sublayer(f"l{i}.norm2")
-                y, ldy = self._feed_forward(i, layer.ff, h, M)
+                y, ldy = self._feed_forward(i, h, M)
                 branches, scale = [(y, ldy, None, 1.0)], w[f"l{i}.ls2"]
             if self._tap is not None:
                 self._sum_norm(x, branches, [], M, col_scale=scale)

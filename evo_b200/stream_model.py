@@ -23,7 +23,7 @@ import torch
 import torch.nn as nn
 
 from . import _lib
-from ._lib import (EPI_NONE, ConvActParams, GatedDeltaParams, GluActParams, LatentDecodeParams, LatentPrepParams, MoeRouteParams, SumNormParams, WindowAttnParams,
+from ._lib import (EPI_GELU_TANH_GATE, EPI_NONE, EPI_SILU_COLS, ConvActParams, GatedDeltaParams, GluActParams, LatentDecodeParams, LatentPrepParams, MoeRouteParams, SumNormParams, WindowAttnParams,
                    check, ptr)
 from .engine import KernelOps
 from .stripedhyena.cache import InferenceParams, RecurrentInferenceParams
@@ -39,11 +39,29 @@ def _round_up(x: int, m: int) -> int:
 class _Packed:
     """A linear layer's weight in the GEMMs' layout: (Np, Kp) bf16, zero rows / columns past (N, K)."""
 
-    def __init__(self, w: torch.Tensor):
+    def __init__(self, w: torch.Tensor, k_tile: int = 64):
         self.N, self.K = w.shape
-        self.Np, self.Kp = _round_up(self.N, 256), _round_up(self.K, 64)
+        self.Np, self.Kp = _round_up(self.N, 256), _round_up(self.K, k_tile)
         self.w = torch.zeros(self.Np, self.Kp, dtype=torch.bfloat16, device=w.device)
         self.w[:self.N, :self.K] = w.to(torch.bfloat16)
+
+
+class _PackedGate(_Packed):
+    """The gate and up weights of a gated feed-forward, (F, K) each, as one linear layer whose rows alternate in runs of RUN, [gate | up]:
+    both halves of a product land in one tile of the GEMM, whose epilogue can then store act(gate) * up, (M, Fp)."""
+    RUN = 128
+
+    def __init__(self, gate: torch.Tensor, up: torch.Tensor):
+        self.F, K = gate.shape
+        self.Fp, self.Kp = _round_up(self.F, self.RUN), _round_up(K, 64)
+        self.N = self.Np = 2 * self.Fp
+        self.K = K
+        self.w = torch.zeros(self.Np, self.Kp, dtype=torch.bfloat16, device=gate.device)
+        runs = self.w.view(self.Fp // self.RUN, 2, self.RUN, self.Kp)
+        for half, src in enumerate((gate, up)):
+            full = torch.zeros(self.Fp, self.Kp, dtype=torch.bfloat16, device=gate.device)
+            full[:self.F, :K] = src.to(torch.bfloat16)
+            runs[:, half] = full.view(-1, self.RUN, self.Kp)
 
 
 class StreamDecoder(KernelOps, nn.Module):
@@ -154,18 +172,38 @@ class StreamDecoder(KernelOps, nn.Module):
     def _dt(self) -> int:
         return 1 if self.act_dtype == torch.float32 else 0
 
-    def _linear(self, a, pk: _Packed, M: int, out=None):
-        """(M, Kp) activations -> (M, Np): rows of A are padded with zeros up to Kp by their producers.  out: rows of a (.., Np) buffer to fill."""
+    @property
+    def _fused(self) -> bool:
+        """Whether linear layers run on the tensor-core GEMMs, whose epilogues can apply an activation."""
+        return not self._dt and self.gemm_path != "simt"
+
+    def _linear(self, a, pk: _Packed, M: int, out=None, silu_cols=0):
+        """(M, Kp) activations -> (M, Np): rows of A are padded with zeros up to Kp by their producers.  out: rows of a (.., Np) buffer to fill.
+        silu_cols: the first columns go through silu in the GEMM's epilogue (only where self._fused; other callers apply it themselves)."""
+        assert not silu_cols or self._fused
+        epi = EPI_SILU_COLS if silu_cols else EPI_NONE
         if out is None:
             out = torch.empty(M, pk.Np, dtype=self.act_dtype, device=a.device)
         if self._dt or self.gemm_path == "simt":
             self._record(f"gemm_simt/{pk.N}x{pk.K}", 2.0 * M * pk.N * pk.K, lambda: check(_lib.lib().evo_gemm_simt(
                 ptr(a), pk.Kp, ptr(pk.w), pk.Kp, ptr(out), pk.Np, M, pk.N, pk.K, self._dt, self._stream()), "evo_gemm_simt"))
         elif M <= 64:
-            self._gemm_smallm(a, pk.w, out, M, pk.Np, pk.Kp, EPI_NONE)
+            self._gemm_smallm(a, pk.w, out, M, pk.Np, pk.Kp, epi, act_cols=silu_cols)
         else:
-            self._gemm(a, pk.w, out, M, pk.Np, pk.Kp, EPI_NONE, variant=2 if M <= 512 else self.gemm_variant)
+            self._gemm(a, pk.w, out, M, pk.Np, pk.Kp, epi, variant=2 if M <= 512 else self.gemm_variant, act_cols=silu_cols)
         return out
+
+    def _gelu_gate(self, h, pk: _PackedGate, M: int):
+        """gelu_tanh(gate h) * (up h) -> (M, Fp), columns past F zero: in the GEMM's epilogue, or by a second kernel behind the fp32 / comparator GEMM."""
+        a = torch.empty(M, pk.Fp, dtype=self.act_dtype, device=h.device)
+        if not self._fused:
+            z = self._linear(h, pk, M)
+            self._glu(z.data_ptr(), z.data_ptr() + pk.RUN * z.element_size(), pk.Np, a, pk.Fp, M, pk.F, 0, interleave=pk.RUN)
+        elif M <= 64:
+            self._gemm_smallm(h, pk.w, a, M, pk.Np, pk.Kp, EPI_GELU_TANH_GATE)
+        else:
+            self._gemm(h, pk.w, a, M, pk.Np, pk.Kp, EPI_GELU_TANH_GATE, ldc=pk.Fp, variant=1 if M <= 512 else self.gemm_variant)
+        return a
 
     # ---- row kernels and mixers shared by several families -----------------------------------------
     def _sum_norm(self, x, branches, outs, rows, gather=None, col_scale=None):
@@ -182,9 +220,9 @@ class StreamDecoder(KernelOps, nn.Module):
         nbytes = rows * cfg.width * (8.0 + esz * (len(branches) + len(outs)))
         self._record("sum_norm", nbytes, lambda: check(_lib.lib().evo_sum_norm(C.byref(p), self._stream()), "evo_sum_norm"))
 
-    def _glu(self, z_ptr, up_ptr, ld, out, ldo, rows, F, act, limit=0.0, slope=1.0, route=None, group=0, n_groups=0, tail_w=0):
+    def _glu(self, z_ptr, up_ptr, ld, out, ldo, rows, F, act, limit=0.0, slope=1.0, route=None, group=0, n_groups=0, tail_w=0, interleave=0):
         """out (rows, ldo) = act(gate) * up [* routing weight of the column's expert] (see evo_glu_act)."""
-        p = GluActParams(gate=z_ptr, up=up_ptr, ld=ld, out=out.data_ptr(), ldo=ldo, rows=rows, F=F, act=act, dtype=self._dt, limit=limit, slope=slope)
+        p = GluActParams(gate=z_ptr, up=up_ptr, ld=ld, out=out.data_ptr(), ldo=ldo, rows=rows, F=F, act=act, dtype=self._dt, limit=limit, slope=slope, interleave=interleave)
         if route is not None:
             p.group_w, p.ldw, p.group, p.n_groups, p.tail_w = route.data_ptr(), route.shape[1], group, n_groups, tail_w
         self._record("glu_act", 3.0 * out.element_size() * rows * F, lambda: check(_lib.lib().evo_glu_act_ex(C.byref(p), self._stream()), "evo_glu_act"))

@@ -60,6 +60,8 @@ enum {
   EVO_EPI_HYENA_STEP = 7, /* evo_gemm_smallm only: the Hyena in-projection (N = 3D, bias) with the decode step of the operator
                              (engine.step_fir + step_iir == evo_hyena_step) applied in the epilogue: a tile is one head's
                              [x2 | x1 | v] rows, C is y (M, D); fir_state / state are updated in place; z is never stored */
+  EVO_EPI_SILU_COLS = 8,  /* C = bf16(n < act_cols ? silu(acc) : acc): projections of which some go through the activation */
+  EVO_EPI_GELU_TANH_GATE = 9, /* like EVO_EPI_GELU_GATE with the tanh form of gelu and one rounding: C[M,N/2] = bf16(gelu_tanh(acc1) * acc2) */
   EVO_EPI_BIAS_ROPE = 6   /* Wqkv projection with the rotary embedding applied where flash_attn applies it
                              (MHA.forward, mha.py:635-648): x = bf16(acc + bias[n]); columns n < rope_cols (q and k,
                              heads of 128) are rotated NeoX-style with the cos/sin row of the token's position
@@ -86,6 +88,7 @@ typedef struct {
    * peer_period = H*128, peer_inner = H/P*128, ldc = 3*peer_inner, peer_row0 = rank * rows.  C is ignored. */
   void* const* c_peers;          /* HOST array of n_c_peers device pointers */
   int n_c_peers; int64_t peer_period, peer_inner, peer_row0;
+  int64_t act_cols;              /* EVO_EPI_SILU_COLS */
 } evo_gemm_params;
 int evo_gemm(const evo_gemm_params* p, void* stream);
 /* Decode-step linear layer (M <= 64 rows): the same C = epilogue(A . W^T) with the same rounding points, as a
@@ -107,6 +110,7 @@ typedef struct {
   void* fir_state; float* state;                 /* (M, 3D, 2) bf16, (M, D, 8, 2) fp32: in/out */
   const void* fir_w; const void* fir_b; const void* Dskip;
   const float* poles; const float* residues;
+  int64_t act_cols;                              /* EVO_EPI_SILU_COLS */
 } evo_gemm_smallm_params;
 size_t evo_gemm_smallm_workspace(int64_t M, int64_t N, int64_t K, int epilogue);
 int evo_gemm_smallm(const evo_gemm_smallm_params* p, void* stream);
@@ -416,6 +420,7 @@ typedef struct {
   void* out; int64_t ldo; int64_t rows; int F, act;
   const float* group_w; int64_t ldw; int group, n_groups, tail_w;
   int dtype; float limit, slope;
+  int interleave;                /* > 0 (a multiple of 4): gate and up share rows of runs [gate | up] of this many columns each; `gate` is the first run, `up` the second */
 } evo_glu_act_params;
 int evo_glu_act_ex(const evo_glu_act_params* p, void* stream);
 
@@ -712,6 +717,7 @@ typedef struct {
   int dtype;
   int B; int64_t L; int H, dk, dv;
   int recurrent;
+  int64_t part_len;             /* tokens per part of a sequence that runs block-wise in parallel parts (0: chosen by the call's size) */
 } evo_decay_scan_params;
 size_t evo_decay_scan_workspace(const evo_decay_scan_params* p);
 int evo_decay_scan_fwd(const evo_decay_scan_params* p, void* workspace, size_t workspace_bytes, void* stream);

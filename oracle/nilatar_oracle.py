@@ -192,3 +192,28 @@ def make_weights(cfg: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
             w[p + "mlp.gate"], w[p + "mlp.up"], w[p + "mlp.down"] = lin(f["ff"], D), lin(f["ff"], D), lin(D, f["ff"])
     w["final.norm"], w["head"] = gain(D), lin(V, D)
     return {k: t.to(torch.bfloat16) for k, t in w.items()}
+
+
+def make_config(kinds=("attention", "latent_attention", "lightning", "shared"), ff=(40, 40, 0, 40), width=64, vocab=101, eps=1e-5, embed_scale=4.0,
+                heads=4, kv_heads=2, dim=16, vdim=12, window=24, scale=0.3,
+                lat_heads=3, lat_dim=8, rot_dim=12, lat_vdim=20, kv_rank=24, q_rank=28, lat_scale=0.25, rot_base=1000.0, scaling=(4.0, 64, 8.0, 1.0),
+                lin_heads=2, lin_dim=12, lin_vdim=24, decay=None) -> dict:
+    """A small configuration; "shared" is an attention layer that reads the keys and values of the last attention layer before it."""
+    decay = decay or [1.0 - 0.5 ** (h + 1) for h in range(lin_heads)]
+    layers, source = [], None
+    for i, kind in enumerate(kinds):
+        if kind == "latent_attention":
+            rot = {"base": rot_base, "dims": rot_dim}
+            if scaling:
+                rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+            m = {"heads": lat_heads, "dim": lat_dim, "rot_dim": rot_dim, "vdim": lat_vdim, "kv_rank": kv_rank, "q_rank": q_rank, "scale": lat_scale, "rot": rot}
+        elif kind == "lightning":
+            m = {"heads": lin_heads, "dim": lin_dim, "vdim": lin_vdim, "decay": list(decay)}
+        else:
+            m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "mask": {"size": window}}
+            if kind == "shared":
+                m["kv_from"] = source
+            else:
+                source = i
+        layers.append({"type": "attention" if kind == "shared" else kind, "mixer": m, "mlp": {"kind": "dense", "ff": ff[i]} if ff[i] else None})
+    return {"architecture": "Nilatar", "vocab": vocab, "width": width, "norm": {"eps": eps}, "embedding": {"scale": embed_scale}, "layers": layers}
