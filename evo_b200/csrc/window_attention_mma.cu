@@ -10,7 +10,12 @@
 // at a time (scores -> softmax -> P.V), so only one 16 x 64 tile of probabilities is live.
 // Head sizes are padded to 16 in shared memory (zero columns); maps x dk <= 256, dv <= 128 and dv % 8 == 0, otherwise the CUDA-core
 // kernel runs.  The tile walk is the CUDA-core kernel's: [0, keep_first), the pooled blocks that the CTA's last query sees, and the
-// union of the CTA's windows.  A soft cap is applied to the fp32 scores before the softmax (tanh from ex2 and a division), and a
+// union of the CTA's windows.
+// One map without kept tokens, pooled blocks, soft cap, bias and head norm -- what most layers ask for -- has a kernel of its own
+// (window_attn_plain_kernel): with one K and one V tile in shared memory three CTAs fit an SM (two with heads wider than 128), a K tile is replaced as soon as its
+// scores are taken and a V tile as soon as it is summed, so that each is on its way while the other is in work and other CTAs fill the
+// waits; the exponents' reference follows the running maximum lazily (weights stay below 2^8).
+// In the general kernel a soft cap is applied to the fp32 scores before the softmax (tanh from ex2 and a division), and a
 // sink enters the denominators at the end; a distance bias is taken off the fp32 scores together with the mask.
 #include "common.cuh"
 #include "mma_sync.cuh"
@@ -317,8 +322,203 @@ __global__ void __launch_bounds__(WARPS * 32) window_attn_mma_kernel(evo_window_
   }
 }
 
+// one map, causal or windowed, optional sink, gate per head or channel.  KSTEPS: 16-column steps of a score product (0: any number)
+template <int NV8, int KSTEPS>
+__global__ void __launch_bounds__(WARPS * 32, KSTEPS > 8 ? 2 : 3) window_attn_plain_kernel(evo_window_attn_params p, int dkp, int vec) {
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  const int st = dkp + 8;                                       // row strides: 16 bytes of padding
+  constexpr int vst = NV8 * 8 + 8;
+  bf16* Qs = reinterpret_cast<bf16*>(smem_raw);                 // [64][st]
+  bf16* Ks = Qs + WARPS * QROWS * st;                           // [KT][st]
+  bf16* Vs = Ks + KT * st;                                      // [KT][vst]
+  const int dk = p.dk, dv = p.dv, ksteps = KSTEPS ? KSTEPS : dkp / 16;
+  const int b = blockIdx.z, h = blockIdx.y, g = h / (p.H / p.G);
+  const int tid = threadIdx.x, w = tid >> 5, lane = tid & 31, qr = lane >> 2, qc = (lane & 3) * 2, mi = lane >> 3;
+  const int64_t pos = p.pos_dev ? (int64_t)*p.pos_dev : p.q_pos0;
+  const int64_t rel0 = (int64_t)(gridDim.x - 1 - blockIdx.x) * (WARPS * QROWS);      // without a window the last queries have the most keys: they go first
+  const int64_t i_lo = pos + rel0, i_hi = pos + min(p.Lq - 1, rel0 + WARPS * QROWS - 1);
+  const bool windowed = p.window > 0;
+  const int64_t key_lo = windowed ? max((int64_t)0, i_lo - p.window + 1) : 0;
+  const int n_tiles = (int)((i_hi - key_lo) / KT) + 1;
+  // everything below counts keys and queries from key_lo, in 32 bits
+  const int n_keys = (int)(i_hi - key_lo) + 1, win = windowed ? (int)min(p.window, (int64_t)1 << 30) : 1 << 30;
+  const int wq = (int)(i_lo - key_lo) + w * QROWS, r0 = wq + qr;      // the warp's first query, the thread's first (the other is 8 further)
+  const bf16* qg = (const bf16*)p.q + ((int64_t)b * p.Lq + rel0) * p.q_tok_stride + (int64_t)h * dk;
+  const bf16* kg = (const bf16*)p.k + (int64_t)b * p.k_batch_stride + key_lo * p.k_tok_stride + (int64_t)g * dk;
+  const bf16* vg = (const bf16*)p.v + (int64_t)b * p.v_batch_stride + key_lo * p.v_tok_stride + (int64_t)g * dv;
+  // rows [0, n) of a tile, `cols` columns of which `live` exist, as asynchronous 16-byte copies (or element by element); a thread's column is fixed where 8 or 16 pieces make a row
+  const auto fetch = [&](bf16* dst, int dst_st, const bf16* src, int64_t ld, int n, int cols, int live) {
+    const int cpr = cols / 8;
+    if (vec) {
+      for (int idx = tid; idx < KT * cpr; idx += WARPS * 32) {
+        const int r = idx / cpr, c = (idx - r * cpr) * 8;
+        const bool on = r < n && c < live;
+        copy16_async(dst + r * dst_st + c, on ? src + r * ld + c : src, on);
+      }
+    } else {
+      for (int idx = tid; idx < KT * cols; idx += WARPS * 32) {
+        const int r = idx / cols, c = idx - r * cols;
+        dst[r * dst_st + c] = r < n && c < live ? src[r * ld + c] : __float2bfloat16_rn(0.f);
+      }
+    }
+    copies_commit();
+  };
+  const auto fetch_k = [&](int t) { const int k0 = t * KT; fetch(Ks, st, kg + (int64_t)k0 * p.k_tok_stride, p.k_tok_stride, min(KT, n_keys - k0), dkp, dk); };
+  const auto fetch_v = [&](int t) { const int k0 = t * KT; fetch(Vs, vst, vg + (int64_t)k0 * p.v_tok_stride, p.v_tok_stride, min(KT, n_keys - k0), NV8 * 8, dv); };
+  fetch(Qs, st, qg, p.q_tok_stride, (int)min((int64_t)(WARPS * QROWS), p.Lq - rel0), dkp, dk);
+  fetch_k(0);
+  fetch_v(0);
+  float O[NV8][4];
+#pragma unroll
+  for (int n = 0; n < NV8; ++n) O[n][0] = O[n][1] = O[n][2] = O[n][3] = 0.f;
+  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;     // references of the exponents (-inf: no key yet) and this lane's part of the sums
+  const float scale2 = p.scale * 1.4426950408889634f;
+  const bf16* qf = Qs + (w * QROWS + (mi & 1) * 8 + (lane & 7)) * st + (mi >> 1) * 8;
+  const bf16* kf = Ks + ((mi >> 1) * 8 + (lane & 7)) * st + (mi & 1) * 8;
+  const bf16* vf = Vs + ((mi & 1) * 8 + (lane & 7)) * vst + (mi >> 1) * 8;
+  for (int t = 0; t < n_tiles; ++t) {
+    const int k0 = t * KT, nk = min(KT, n_keys - k0);
+    copies_wait<1>();                                  // the K tile (and the queries); the V tile may still be on its way
+    __syncthreads();
+    // does any row of the warp see any key of the tile, do all rows see all of it
+    const bool some = k0 <= wq + QROWS - 1 && wq - (k0 + nk - 1) < win;
+    const bool full = nk == KT && k0 + KT - 1 <= wq && wq + QROWS - 1 - k0 < win;
+    float P[KT / 8][4];
+    if (some) {
+#pragma unroll
+      for (int n = 0; n < KT / 8; ++n) P[n][0] = P[n][1] = P[n][2] = P[n][3] = 0.f;
+#pragma unroll 4
+      for (int ks = 0; ks < ksteps; ++ks) {
+        uint32_t a[4];
+        ldmatrix_x4(a, qf + ks * 16);
+#pragma unroll
+        for (int n = 0; n < KT / 8; n += 2) {
+          uint32_t f[4];
+          ldmatrix_x4(f, kf + n * 8 * st + ks * 16);
+          mma_bf16(P[n], a, f[0], f[1]);
+          mma_bf16(P[n + 1], a, f[2], f[3]);
+        }
+      }
+    }
+    __syncthreads();                                   // the K tile has been read by every warp
+    if (t + 1 < n_tiles) fetch_k(t + 1); else copies_commit();
+    if (some) {
+      float mx0 = -INFINITY, mx1 = -INFINITY;
+      if (!full) {
+#pragma unroll
+        for (int n = 0; n < KT / 8; ++n)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            const int d = r0 + (c >> 1) * 8 - (k0 + n * 8 + qc + (c & 1));         // distance; keys past the tile's last one lie behind every query
+            if (d < 0 || d >= win) P[n][c] = -INFINITY;
+          }
+      }
+#pragma unroll
+      for (int n = 0; n < KT / 8; ++n) { mx0 = fmaxf(mx0, fmaxf(P[n][0], P[n][1])); mx1 = fmaxf(mx1, fmaxf(P[n][2], P[n][3])); }
+      mx0 = quad_max(mx0) * scale2; mx1 = quad_max(mx1) * scale2;
+      const bool grow = (mx0 > m0 + 8.f) || (mx1 > m1 + 8.f);                         // also true for a row's first keys (m = -inf)
+      if (__any_sync(0xffffffffu, grow)) {
+        const float n0 = fmaxf(m0, mx0), n1 = fmaxf(m1, mx1);
+        const float c0 = m0 == -INFINITY ? 0.f : ex2(m0 - n0), c1 = m1 == -INFINITY ? 0.f : ex2(m1 - n1);
+        m0 = n0; m1 = n1;
+        l0 *= c0; l1 *= c1;
+#pragma unroll
+        for (int n = 0; n < NV8; ++n) { O[n][0] *= c0; O[n][1] *= c0; O[n][2] *= c1; O[n][3] *= c1; }
+      }
+      const float ref0 = m0 == -INFINITY ? 0.f : m0, ref1 = m1 == -INFINITY ? 0.f : m1;
+#pragma unroll
+      for (int n = 0; n < KT / 8; ++n) {
+        P[n][0] = ex2(fmaf(P[n][0], scale2, -ref0)); P[n][1] = ex2(fmaf(P[n][1], scale2, -ref0));
+        P[n][2] = ex2(fmaf(P[n][2], scale2, -ref1)); P[n][3] = ex2(fmaf(P[n][3], scale2, -ref1));
+        l0 += P[n][0] + P[n][1]; l1 += P[n][2] + P[n][3];
+      }
+    }
+    copies_wait<1>();                                  // the V tile; the next K tile may still be on its way
+    __syncthreads();
+    if (some) {
+#pragma unroll
+      for (int kk = 0; kk < KT / 16; ++kk) {
+        uint32_t ah[4], al[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {                  // rows (qr, qr + 8) x keys (qc.., qc + 8..)
+          const float x = P[2 * kk + (e >> 1)][(e & 1) * 2], y = P[2 * kk + (e >> 1)][(e & 1) * 2 + 1];
+          ah[e] = pack_bf16(x, y);
+          al[e] = pack_bf16(x - bf_lo(ah[e]), y - bf_hi(ah[e]));
+        }
+#pragma unroll
+        for (int n = 0; n < NV8; n += 2) {
+          uint32_t f[4];
+          ldmatrix_x4_trans(f, vf + kk * 16 * vst + n * 8);
+          mma_bf16(O[n], ah, f[0], f[1]); mma_bf16(O[n + 1], ah, f[2], f[3]);
+          mma_bf16(O[n], al, f[0], f[1]); mma_bf16(O[n + 1], al, f[2], f[3]);
+        }
+      }
+    }
+    if (t + 1 < n_tiles) {
+      __syncthreads();                                 // the V tile has been read by every warp
+      fetch_v(t + 1);
+    }
+  }
+  copies_wait<0>();
+  l0 = quad_sum(l0); l1 = quad_sum(l1);
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int64_t rel = rel0 + w * QROWS + qr + 8 * half;
+    if (rel >= p.Lq) continue;
+    const float m = half ? m1 : m0, l = half ? l1 : l0;
+    float mul = 1.f / l;
+    if (p.sink) {                                      // e^sink joins the denominator
+      const float sk = __bfloat162float(((const bf16*)p.sink)[h]) * 1.4426950408889634f, mx = fmaxf(m, sk), num = ex2(m - mx);
+      mul = num / fmaf(l, num, ex2(sk - mx));
+    }
+    const int64_t row = (int64_t)b * p.Lq + rel;
+    const bf16* grow = p.gate ? (const bf16*)p.gate + row * p.gate_tok_stride + (p.gate_per_head ? h : (int64_t)h * dv) : nullptr;
+    if (grow && p.gate_per_head) mul *= 1.f / (1.f + expf(-__bfloat162float(*grow)));
+    const bool chan = grow && !p.gate_per_head, pairs = chan && ((uintptr_t)grow & 3) == 0;
+    bf16* orow = (bf16*)p.out + row * p.ldo + (int64_t)h * dv;
+#pragma unroll
+    for (int n = 0; n < NV8; ++n) {
+      const int ch = n * 8 + qc;
+      if (ch < dv) {                                   // dv is even: the pair (ch, ch + 1) is inside the head
+        float v0 = O[n][2 * half] * mul, v1 = O[n][2 * half + 1] * mul;
+        if (chan) {
+          float g0, g1;
+          if (pairs) { const uint32_t u = *reinterpret_cast<const uint32_t*>(grow + ch); g0 = bf_lo(u); g1 = bf_hi(u); }
+          else { g0 = __bfloat162float(grow[ch]); g1 = __bfloat162float(grow[ch + 1]); }
+          v0 *= __fdividef(1.f, 1.f + __expf(-g0));
+          v1 *= __fdividef(1.f, 1.f + __expf(-g1));
+        }
+        orow[ch] = __float2bfloat16_rn(v0);
+        orow[ch + 1] = __float2bfloat16_rn(v1);
+      }
+    }
+    if (h == p.H - 1)
+      for (int64_t c = (int64_t)p.H * dv + (lane & 3); c < p.ldo; c += 4) ((bf16*)p.out)[row * p.ldo + c] = __float2bfloat16_rn(0.f);
+  }
+}
+
+template <int NV8, int KSTEPS>
+int launch_plain(const evo_window_attn_params* p, cudaStream_t st) {
+  const int dkp = (p->dk + 15) / 16 * 16;
+  auto a16 = [](const void* q) { return ((uintptr_t)q & 15) == 0; };
+  const int vec = p->dk % 8 == 0 && p->dv % 8 == 0 && p->q_tok_stride % 8 == 0 && p->k_tok_stride % 8 == 0 && p->v_tok_stride % 8 == 0 &&
+                  p->k_batch_stride % 8 == 0 && p->v_batch_stride % 8 == 0 && a16(p->q) && a16(p->k) && a16(p->v);
+  const size_t smem = sizeof(bf16) * ((size_t)(WARPS * QROWS + KT) * (dkp + 8) + (size_t)KT * (NV8 * 8 + 8));
+  auto kern = window_attn_plain_kernel<NV8, KSTEPS>;
+  if (smem > 48 * 1024) EVO_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  kern<<<dim3((unsigned)((p->Lq + WARPS * QROWS - 1) / (WARPS * QROWS)), p->H, p->B), WARPS * 32, smem, st>>>(*p, dkp, vec);
+  return check_launch("evo_window_attn_fwd");
+}
+
 template <int NV8, int NM>
 int launch(const evo_window_attn_params* p, cudaStream_t st) {
+  if (NM == 1 && p->keep_first <= 0 && p->pool <= 0 && !(p->softcap > 0.f) && !p->dist_r1 && !p->head_norm && p->scale > 0.f && p->q_pos0 + p->Lq < (1 << 30)) {
+    // the usual sizes with the number of score steps known to the compiler
+    if (NV8 == 16 && p->dk == 128) return launch_plain<NV8, NV8 == 16 ? 8 : 0>(p, st);
+    if (NV8 == 16 && p->dk == 192) return launch_plain<NV8, NV8 == 16 ? 12 : 0>(p, st);
+    if (NV8 == 8 && p->dk == 64) return launch_plain<NV8, NV8 == 8 ? 4 : 0>(p, st);
+    return launch_plain<NV8, 0>(p, st);
+  }
   const int dkp = (p->dk + 15) / 16 * 16;
   const int qst = NM * dkp + 8, kst = NM * dkp + 8, vst = NV8 * 8 + 8;
   // two K/V buffers (the next tile is fetched while the current one is in work) as long as two CTAs still fit an SM's shared memory

@@ -278,6 +278,58 @@ def test_sink_windows_with_a_gate_per_channel(H, G, dk, dv, window):
         _close(torch.cat(outs, 0), want, tol, f"{dtype}, {rows} rows a call")
 
 
+# heads, key heads, dk, dv, window, rows, first position: one tile, a tile and a bit, several pairs of tiles; windows of one position, at and
+# around a key tile, longer than the sequence; every count of 64-column halves, head sizes that fill none of them
+PROMPT_SHAPES = [(2, 1, 64, 64, 0, 128, 0), (2, 2, 128, 128, 0, 300, 77), (1, 1, 192, 128, 0, 257, 3), (3, 1, 192, 40, 200, 400, 130), (4, 2, 48, 48, 136, 310, 0), (2, 1, 128, 128, 1, 260, 5),
+                 (2, 2, 64, 128, 128, 520, 64), (2, 1, 72, 72, 129, 385, 1), (1, 1, 136, 8, 127, 300, 900), (2, 2, 8, 16, 40, 140, 0), (2, 1, 128, 64, 5000, 200, 10), (1, 1, 128, 128, 300, 700, 411),
+                 (3, 3, 80, 104, 90, 200, 17), (2, 1, 176, 120, 0, 150, 60), (5, 5, 16, 8, 33, 129, 2)]
+
+
+@pytest.mark.parametrize("H,G,dk,dv,window,L,pos0", PROMPT_SHAPES, ids=lambda v: str(v))
+def test_prompt_attention_on_the_tensor_cores(H, G, dk, dv, window, L, pos0):
+    """Two sequences in one call, each with cache rows of its own; the rows behind the last position hold NaNs; with and without sink, a
+    gate per channel, per head and none."""
+    g = torch.Generator().manual_seed(dk + L)
+    B, T, lib = 2, pos0 + L, _lib.lib()
+    cw, rows = G * (dk + dv), T + 5
+    q, kv = _bf(torch.randn(B, L, H, dk, generator=g)), torch.full((B, rows, cw), float("nan"))
+    kv[:, :T] = torch.randn(B, T, cw, generator=g)
+    kv, gate, sink = _bf(kv), _bf(torch.randn(B * L, H * dv, generator=g)), _bf(torch.randn(H, generator=g) * 2)
+    scale, ldo = 1.4 / math.sqrt(dk), (H * dv + 63) // 64 * 64
+    qd, kvd, gd, sd = q.to(DEV), kv.to(DEV), gate.to(DEV), sink.to(DEV)
+    k, v = kv[:, :T, :G * dk].double().view(B, T, G, dk), kv[:, :T, G * dk:].double().view(B, T, G, dv)
+    for with_sink, per_head in ((True, False), (False, True), (False, None)):
+        want = torch.stack([O.softmax_attention(q[b].double(), k[b], v[b], scale, window, sink.double() if with_sink else None, pos0) for b in range(B)]).reshape(B * L, H * dv)
+        if per_head is not None:
+            s = torch.sigmoid(gate.double())
+            want = want * (s[:, :H].repeat_interleave(dv, 1) if per_head else s)
+        out = torch.full((B * L, ldo), 5.0, dtype=B16, device=DEV)
+        p = WindowAttnParams(q=qd.data_ptr(), q_tok_stride=H * dk, k=kvd.data_ptr(), v=kvd.data_ptr() + 2 * G * dk, k_tok_stride=cw, v_tok_stride=cw, k_batch_stride=rows * cw,
+                             v_batch_stride=rows * cw, gate=gd.data_ptr() if per_head is not None else None, gate_tok_stride=H * dv, gate_per_head=int(bool(per_head)),
+                             out=out.data_ptr(), ldo=ldo, dtype=0, B=B, Lq=L, H=H, G=G, dk=dk, dv=dv, n_maps=1, q_pos0=pos0, window=window, scale=scale,
+                             sink=sd.data_ptr() if with_sink else None)
+        check(lib.evo_window_attn_fwd(C.byref(p), _stream()))
+        _close(out[:, :H * dv], want, 6e-3, f"sink {with_sink}, gate per head {per_head}")
+        assert (out[:, H * dv:] == 0).all()
+
+
+def test_prompt_attention_weights_keep_sixteen_bits():
+    """Equal scores over thousands of keys with values of one sign: weights rounded to bf16 would shift every output by up to 2^-9."""
+    g = torch.Generator().manual_seed(2)
+    T, dk, dv = 2100, 64, 64
+    q, k, v = torch.zeros(T, 1, dk), torch.zeros(T, 1, dk), 1.0 + torch.rand(T, 1, dv, generator=g)
+    q[..., 0], k[..., 0] = 1.0, torch.randn(T, 1, generator=g) * 0.3
+    q, k, v = _bf(q), _bf(k), _bf(v)
+    want = O.softmax_attention(q.double(), k.double(), v.double(), 1.0).reshape(T, dv)
+    out = torch.empty(T, dv, dtype=B16, device=DEV)
+    qd, kd, vd = q.to(DEV), k.to(DEV), v.to(DEV)
+    p = WindowAttnParams(q=qd.data_ptr(), q_tok_stride=dk, k=kd.data_ptr(), v=vd.data_ptr(), k_tok_stride=dk, v_tok_stride=dv, k_batch_stride=T * dk, v_batch_stride=T * dv,
+                         out=out.data_ptr(), ldo=dv, dtype=0, B=1, Lq=T, H=1, G=1, dk=dk, dv=dv, n_maps=1, scale=1.0)
+    check(_lib.lib().evo_window_attn_fwd(C.byref(p), _stream()))
+    assert torch.equal(out.cpu(), _bf(want)) or ((out.double().cpu() - want).abs() <= 2.0 ** -8 * 1.02).all()
+    assert (out.double().cpu() - _bf(want).double()).ne(0).double().mean() < 0.02      # almost every output is the correctly rounded one
+
+
 # ------------------------------------------------------------------ each mixer alone
 def _one_layer(kind, T, seed, **sizes):
     cfg = O.make_config(kinds=(kind,), ff=(0,), vocab=61, **sizes)
