@@ -202,7 +202,9 @@ __device__ __forceinline__ void update_state(float (&S)[MT][8][4], const bf16* K
         split_pack(bf_lo(f[2]) * p8, bf_hi(f[2]) * p9, ah[2], al[2]);
         split_pack(bf_lo(f[3]) * p8, bf_hi(f[3]) * p9, ah[3], al[3]);
 #pragma unroll
-        for (int n = 0; n < 8; ++n) { mma_bf16(S[m][n], ah, bv[n][0], bv[n][1]); mma_bf16(S[m][n], al, bv[n][0], bv[n][1]); }
+        for (int n = 0; n < 8; ++n) mma_bf16(S[m][n], ah, bv[n][0], bv[n][1]);       // products into the same sums stay eight apart
+#pragma unroll
+        for (int n = 0; n < 8; ++n) mma_bf16(S[m][n], al, bv[n][0], bv[n][1]);
       }
     }
   }
@@ -364,10 +366,13 @@ __global__ void __launch_bounds__(128 * CG) decay_block_kernel(BlockArgs a) {
 #pragma unroll
         for (int n = 0; n < 8; n += 2) {
           uint32_t f[4];
-          const int at = (ks * 16 + (mi & 1) * 8 + (lane & 7)) * VST + cg * 64 + (n + (mi >> 1)) * 8;
-          ldmatrix_x4_trans(f, Sh + at);
+          ldmatrix_x4_trans(f, Sh + (ks * 16 + (mi & 1) * 8 + (lane & 7)) * VST + cg * 64 + (n + (mi >> 1)) * 8);
           mma_bf16(O[n], q, f[0], f[1]); mma_bf16(O[n + 1], q, f[2], f[3]);
-          ldmatrix_x4_trans(f, Sl + at);
+        }
+#pragma unroll
+        for (int n = 0; n < 8; n += 2) {
+          uint32_t f[4];
+          ldmatrix_x4_trans(f, Sl + (ks * 16 + (mi & 1) * 8 + (lane & 7)) * VST + cg * 64 + (n + (mi >> 1)) * 8);
           mma_bf16(O[n], q, f[0], f[1]); mma_bf16(O[n + 1], q, f[2], f[3]);
         }
       }
@@ -401,11 +406,12 @@ __global__ void __launch_bounds__(128 * CG) decay_block_kernel(BlockArgs a) {
         split_pack(P[2 * kk + 1][0], P[2 * kk + 1][1], ah[2], al[2]);
         split_pack(P[2 * kk + 1][2], P[2 * kk + 1][3], ah[3], al[3]);
 #pragma unroll
-        for (int n = 0; n < 8; n += 2) {
-          uint32_t f[4];
+        for (int n = 0; n < 8; n += 4) {
+          uint32_t f[4], e[4];
           ldmatrix_x4_trans(f, Vs + (kk * 16 + (mi & 1) * 8 + (lane & 7)) * VST + cg * 64 + (n + (mi >> 1)) * 8);
-          mma_bf16(O[n], ah, f[0], f[1]); mma_bf16(O[n], al, f[0], f[1]);
-          mma_bf16(O[n + 1], ah, f[2], f[3]); mma_bf16(O[n + 1], al, f[2], f[3]);
+          ldmatrix_x4_trans(e, Vs + (kk * 16 + (mi & 1) * 8 + (lane & 7)) * VST + cg * 64 + (n + 2 + (mi >> 1)) * 8);
+          mma_bf16(O[n], ah, f[0], f[1]); mma_bf16(O[n + 1], ah, f[2], f[3]); mma_bf16(O[n + 2], ah, e[0], e[1]); mma_bf16(O[n + 3], ah, e[2], e[3]);
+          mma_bf16(O[n], al, f[0], f[1]); mma_bf16(O[n + 1], al, f[2], f[3]); mma_bf16(O[n + 2], al, e[0], e[1]); mma_bf16(O[n + 3], al, e[2], e[3]);
         }
       }
 #pragma unroll

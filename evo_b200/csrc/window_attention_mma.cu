@@ -446,11 +446,14 @@ __global__ void __launch_bounds__(WARPS * 32, KSTEPS > 8 ? 2 : 3) window_attn_pl
           al[e] = pack_bf16(x - bf_lo(ah[e]), y - bf_hi(ah[e]));
         }
 #pragma unroll
-        for (int n = 0; n < NV8; n += 2) {
-          uint32_t f[4];
+        for (int n = 0; n < NV8; n += 4) {             // products into the same sums stay four apart
+          uint32_t f[4], e[4];
           ldmatrix_x4_trans(f, vf + kk * 16 * vst + n * 8);
+          if (n + 2 < NV8) ldmatrix_x4_trans(e, vf + kk * 16 * vst + (n + 2) * 8);
           mma_bf16(O[n], ah, f[0], f[1]); mma_bf16(O[n + 1], ah, f[2], f[3]);
+          if (n + 2 < NV8) { mma_bf16(O[n + 2], ah, e[0], e[1]); mma_bf16(O[n + 3], ah, e[2], e[3]); }
           mma_bf16(O[n], al, f[0], f[1]); mma_bf16(O[n + 1], al, f[2], f[3]);
+          if (n + 2 < NV8) { mma_bf16(O[n + 2], al, e[0], e[1]); mma_bf16(O[n + 3], al, e[2], e[3]); }
         }
       }
     }

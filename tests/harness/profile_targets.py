@@ -157,4 +157,27 @@ elif what in ("gagotar", "gagotar_step"):
             d["mha"].seqlen_offset = d["hyena"].seqlen_offset = ctx + t
             lg, _ = model(nxt, inference_params_dict=d)
     torch.cuda.synchronize()
+elif what in ("nilatar", "nilatar_step"):
+    # a 3-layer Nilatar model (windowed sink attention, latent attention, constant-decay linear attention) at width 2048: one prompt of 2 x 4096
+    # tokens ("nilatar") or single-token steps of 16 sequences behind 2048 tokens ("nilatar_step")
+    from evo_b200.nilatar import Nilatar, NilatarConfig
+    layers = [{"type": "attention", "mlp": {"kind": "dense", "ff": 5632}, "mixer": {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024}}},
+              {"type": "latent_attention", "mlp": None, "mixer": {"heads": 16, "dim": 64, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": 768, "scale": 128 ** -0.5,
+                                                                  "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}},
+              {"type": "lightning", "mlp": None, "mixer": {"heads": 16, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-2.0 - 6.0 * h / 16) for h in range(16)]}}]
+    nc = {"architecture": "Nilatar", "vocab": 512, "width": 2048, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "layers": layers}
+    model = Nilatar(NilatarConfig.from_dict(nc)).init_random(0, device=dev)
+    if what == "nilatar":
+        ids = torch.randint(0, 512, (2, 4096), device=dev)
+        for _ in range(2):
+            model(ids)
+    else:
+        B, ctx = 16, 2048
+        d = model.initialize_inference_params(max_seqlen=ctx + 64, max_batch_size=B)
+        lg, d = model(torch.randint(0, 512, (B, ctx), device=dev), inference_params_dict=d)
+        nxt = lg[:, -1].argmax(-1, keepdim=True)
+        for t in range(3):
+            d["mha"].seqlen_offset = d["hyena"].seqlen_offset = ctx + t
+            lg, _ = model(nxt, inference_params_dict=d)
+    torch.cuda.synchronize()
 print("done", what)
